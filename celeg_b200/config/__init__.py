@@ -18,6 +18,9 @@ from .naselorn_arch import build_naselorn_spec
 from .liverax import LiveraxConfig
 from . import liverax_arch as _liverax_arch  # registers "Liverax"
 from .liverax_arch import build_liverax_spec
+from .kodupel import KodupelConfig
+from . import kodupel_arch as _kodupel_arch  # registers "Kodupel"
+from .kodupel_arch import build_kodupel_spec
 
 __all__ = [
     "Architecture", "ConfigError", "UnknownArchitectureError", "ExecutionEntry", "LayerSpec",
@@ -25,5 +28,5 @@ __all__ = [
     "known_architectures", "read_config_json", "register_architecture", "CONV",
     "FULL_ATTENTION", "Lfm2Config", "build_lfm2_spec", "RamosunConfig", "build_ramosun_spec",
     "KedesunConfig", "build_kedesun_spec", "NaselornConfig", "build_naselorn_spec",
-    "LiveraxConfig", "build_liverax_spec",
+    "LiveraxConfig", "build_liverax_spec", "KodupelConfig", "build_kodupel_spec",
 ]

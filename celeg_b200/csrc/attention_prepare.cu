@@ -3,17 +3,20 @@
 //
 //   1. the biases of q, k and v (optional);
 //   2. one RMS norm over the whole q projection and one over the whole k projection, each with a weight as wide as
-//      the projection (optional): x / sqrt(mean(x^2) + eps) * w, the mean over all heads' entries together;
-//   3. the rotation of the first `rotary_dim` entries of every q and k head in pairs (i, i + rotary_dim / 2) by the
-//      angle position * frequency_i (optional; frequencies come from the host, already divided by what the
-//      configuration scales them by);
+//      the projection (optional): x / sqrt(mean(x^2) + eps) * w, the mean over all heads' entries together; or the
+//      same per head with one weight of a head's size for all heads (`norm_per_head`);
+//   3. the rotation of the first `rotary_dim` entries of every q and k head in pairs (i, i + rotary_dim / 2), or of
+//      neighbours (2i, 2i + 1) (`interleaved`), by the angle position * frequency_i, cosine and sine times `magnitude`
+//      (optional; frequencies come from the host, already scaled as the configuration says);
 //   4. a factor on q that grows with the position: 1 + coef * ln(floor((position + 1) / every) + 1) (optional);
 //   5. the blend of the values with those an earlier layer made of the same token: v <- (1 - lam) v + lam v_first
 //      (`blend` 2), or the note of this layer's values for later layers (`blend` 1: v_first <- v);
+//   6. every value head divided by its root mean square, x / sqrt(mean(x^2) + eps), no weight (`unit_values`);
 //
 // rounds once, and writes q to its buffer and k and v to the token's place in the paged cache. A stored head may be
 // wider than the projected one (keys and values brought to one size for kernels that want them alike): the tail is
-// zeros, which change no score and no result.
+// zeros, which change no score and no result. Without caches the rows hold queries alone (a layer that reads another
+// layer's keys and values).
 #include "common.cuh"
 
 namespace celeg_b200 {
@@ -23,7 +26,10 @@ struct QkvPrepareArgs {
     const float* bias;                        // q, k and v biases one after the other, or null
     const float* q_norm_w; const float* k_norm_w;      // [q width], [k width], or null (both or none)
     float norm_eps;
+    int norm_per_head;                        // the norms' weights are [head_dim] and each head has a mean of its own
+    int unit_values; float value_eps;
     const float* frequencies; int rotary_dim; // [rotary_dim / 2] or null
+    int interleaved; float magnitude;
     float temp_coef; int temp_every;          // every <= 0: no factor
     int blend; float lam; float* first_values; int first_stride;     // [tokens, kv_heads * value_dim] float32
     void* q_out; int q_stride;                // queries in the activation type, head h at h * key_store
@@ -97,15 +103,15 @@ __global__ void qkv_prepare_kernel(const QkvPrepareArgs p) {
     }
     if (first_row)
         for (int i = threadIdx.x; i < v_width; i += blockDim.x) first_s[i] = first_row[i];
-    const int page = p.block_table[(size_t)span * p.table_stride + pos / p.page_tokens];
+    const int page = p.kv_heads > 0 ? p.block_table[(size_t)span * p.table_stride + pos / p.page_tokens] : 0;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
         sincosf((float)pos * p.frequencies[i], &s, &c);
-        turn[i] = c;
-        turn[half + i] = s;
+        turn[i] = c * p.magnitude;
+        turn[half + i] = s * p.magnitude;
     }
     float q_factor = 1.0f, k_factor = 1.0f;
-    if (p.q_norm_w) {
+    if (p.q_norm_w && !p.norm_per_head) {
         q_factor = 1.0f / sqrtf(block_sum(q_squares, scratch) / (float)q_width + p.norm_eps);
         k_factor = 1.0f / sqrtf(block_sum(k_squares, scratch) / (float)k_width + p.norm_eps);
     }
@@ -120,22 +126,28 @@ __global__ void qkv_prepare_kernel(const QkvPrepareArgs p) {
         const bool is_q = unit < p.q_heads;
         if (!is_q && page < 0) continue;
         const float* head = qk + (size_t)unit * p.head_dim;
-        const float* weight = !p.q_norm_w ? nullptr
-                              : (is_q ? p.q_norm_w + (size_t)unit * p.head_dim
-                                      : p.k_norm_w + (size_t)(unit - p.q_heads) * p.head_dim);
-        const float factor = is_q ? q_factor : k_factor;
+        const float* weight = is_q ? p.q_norm_w : p.k_norm_w;
+        float factor = is_q ? q_factor : k_factor;
+        if (weight && p.norm_per_head) {
+            float squares = 0.0f;
+            for (int e = lane; e < p.head_dim; e += 32) squares += head[e] * head[e];
+            factor = 1.0f / sqrtf(warp_sum(squares) / (float)p.head_dim + p.norm_eps);
+        } else if (weight) {
+            weight += (size_t)(is_q ? unit : unit - p.q_heads) * p.head_dim;
+        }
         const float after = is_q ? temperature : 1.0f;
         A* dst = is_q ? q_row + (size_t)unit * p.key_store
                       : static_cast<A*>(p.k_cache) + (long long)page * p.page_stride +
                             ((long long)(unit - p.q_heads) * p.page_tokens + in_page) * p.key_store;
         for (int i = lane; i < half; i += 32) {
-            float u = head[i] * factor, v = head[i + half] * factor;
+            const int first = p.interleaved ? 2 * i : i, second = p.interleaved ? 2 * i + 1 : i + half;
+            float u = head[first] * factor, v = head[second] * factor;
             if (weight) {
-                u *= weight[i];
-                v *= weight[i + half];
+                u *= weight[first];
+                v *= weight[second];
             }
-            dst[i] = from_float<A>((u * turn[i] - v * turn[half + i]) * after);
-            dst[i + half] = from_float<A>((v * turn[i] + u * turn[half + i]) * after);
+            dst[first] = from_float<A>((u * turn[i] - v * turn[half + i]) * after);
+            dst[second] = from_float<A>((v * turn[i] + u * turn[half + i]) * after);
         }
         for (int e = 2 * half + lane; e < p.head_dim; e += 32)
             dst[e] = from_float<A>(head[e] * factor * (weight ? weight[e] : 1.0f) * after);
@@ -145,13 +157,26 @@ __global__ void qkv_prepare_kernel(const QkvPrepareArgs p) {
         A* dst = page < 0 ? nullptr
                           : static_cast<A*>(p.v_cache) + (long long)page * p.value_page_stride +
                                 ((long long)unit * p.page_tokens + in_page) * p.value_store;
+        auto blended = [&](int column) {
+            const float v = qk[qk_width + column];
+            return p.blend == 2 ? (1.0f - p.lam) * v + p.lam * first_s[column] : v;
+        };
+        float unit_factor = 1.0f;
+        if (p.unit_values) {
+            float squares = 0.0f;
+            for (int e = lane; e < p.value_dim; e += 32) {
+                const float v = blended(unit * p.value_dim + e);
+                squares += v * v;
+            }
+            unit_factor = 1.0f / sqrtf(warp_sum(squares) / (float)p.value_dim + p.value_eps);
+        }
         for (int e = lane; e < p.value_store; e += 32) {
             float v = 0.0f;
             if (e < p.value_dim) {
                 const int column = unit * p.value_dim + e;
-                v = qk[qk_width + column];
+                v = blended(column);
                 if (p.blend == 1) p.first_values[(size_t)t * p.first_stride + column] = v;
-                if (p.blend == 2) v = (1.0f - p.lam) * v + p.lam * first_s[column];
+                v *= unit_factor;
             }
             if (dst) dst[e] = from_float<A>(v);
         }
@@ -163,21 +188,25 @@ __global__ void qkv_prepare_kernel(const QkvPrepareArgs p) {
 using namespace celeg_b200;
 
 CELEG_API int celeg_qkv_prepare(const float* proj, int proj_stride, const float* bias, const float* q_norm_w,
-                                const float* k_norm_w, float norm_eps, const float* frequencies, int rotary_dim,
+                                const float* k_norm_w, float norm_eps, int norm_per_head, int unit_values, float value_eps,
+                                const float* frequencies, int rotary_dim, int interleaved, float magnitude,
                                 float temp_coef, int temp_every, int blend, float lam, float* first_values,
                                 int first_stride, void* q_out, int q_stride, const int* positions, const int* token_span,
                                 const int* block_table, int table_stride, void* k_cache, void* v_cache,
                                 long long page_stride, long long value_page_stride, int tokens, int q_heads, int kv_heads,
                                 int head_dim, int value_dim, int key_store, int value_store, int page_tokens,
                                 int* error_flag, int act_dtype, cudaStream_t stream) {
-    CELEG_REQUIRE(tokens >= 0 && q_heads > 0 && kv_heads > 0 && head_dim > 0 && value_dim > 0 && page_tokens > 0 &&
+    // (no caches: the rows hold queries alone, kv_heads is 0)
+    CELEG_REQUIRE((kv_heads > 0) == (k_cache != nullptr) && (kv_heads > 0) == (v_cache != nullptr),
+                  "qkv_prepare: %d key heads %s caches", kv_heads, k_cache ? "with" : "without");
+    CELEG_REQUIRE(tokens >= 0 && q_heads > 0 && kv_heads >= 0 && head_dim > 0 && value_dim > 0 && page_tokens > 0 &&
                   key_store >= head_dim && value_store >= value_dim && q_stride >= q_heads * key_store &&
                   proj_stride >= q_heads * head_dim + kv_heads * (head_dim + value_dim),
                   "qkv_prepare: invalid sizes tokens=%d q_heads=%d kv_heads=%d head_dim=%d value_dim=%d stored %d / %d "
                   "strides %d / %d", tokens, q_heads, kv_heads, head_dim, value_dim, key_store, value_store, proj_stride,
                   q_stride);
-    CELEG_REQUIRE((q_norm_w == nullptr) == (k_norm_w == nullptr) && (!q_norm_w || norm_eps > 0.0f),
-                  "qkv_prepare: the whole-projection norm needs both weights and a positive eps");
+    CELEG_REQUIRE(((q_norm_w == nullptr) == (k_norm_w == nullptr) || kv_heads == 0) && (!q_norm_w || norm_eps > 0.0f) &&
+                  (!unit_values || value_eps > 0.0f), "qkv_prepare: the norms need both weights and a positive eps");
     CELEG_REQUIRE(!frequencies || (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= head_dim),
                   "qkv_prepare: %d rotated dimensions of a head of %d", rotary_dim, head_dim);
     CELEG_REQUIRE(blend == 0 || ((blend == 1 || blend == 2) && first_values && first_stride >= kv_heads * value_dim),
@@ -188,9 +217,9 @@ CELEG_API int celeg_qkv_prepare(const float* proj, int proj_stride, const float*
     const size_t first_floats = blend == 2 ? (((size_t)kv_heads * value_dim + 3) & ~(size_t)3) : 0;
     const size_t smem = (row_floats + first_floats + (frequencies ? rotary_dim : 0)) * sizeof(float);
     CELEG_REQUIRE(smem <= 200 * 1024, "qkv_prepare: a row of %zu bytes exceeds a block's shared memory", smem);
-    const QkvPrepareArgs args = {proj, proj_stride, bias, q_norm_w, k_norm_w, norm_eps, frequencies, rotary_dim,
-                                 temp_coef, temp_every, blend, lam, first_values, first_stride, q_out, q_stride,
-                                 positions, token_span, block_table, table_stride, k_cache, v_cache, page_stride,
+    const QkvPrepareArgs args = {proj, proj_stride, bias, q_norm_w, k_norm_w, norm_eps, norm_per_head,
+                                 unit_values, value_eps, frequencies, rotary_dim, interleaved, magnitude, temp_coef,
+                                 temp_every, blend, lam, first_values, first_stride, q_out, q_stride, positions, token_span, block_table, table_stride, k_cache, v_cache, page_stride,
                                  value_page_stride, q_heads, kv_heads, head_dim, value_dim, key_store, value_store,
                                  page_tokens, error_flag};
     cudaError_t status = cudaSuccess;

@@ -59,15 +59,30 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 }
 
 // Element-wise activations by code (the feed-forward parts name one): 0 the exact GELU (erf), 1 the tanh GELU, 2 SiLU,
-// 3 the square of ReLU, 4 ReLU.
-enum Activation : int { kGeluErf = 0, kGeluTanh = 1, kSilu = 2, kSquaredRelu = 3, kRelu = 4 };
+// 3 the square of ReLU, 4 ReLU, 5 tanh.
+enum Activation : int { kGeluErf = 0, kGeluTanh = 1, kSilu = 2, kSquaredRelu = 3, kRelu = 4, kTanh = 5 };
 
 __device__ __forceinline__ float activate(float z, int kind) {
     if (kind == kGeluErf) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
     if (kind == kGeluTanh) return 0.5f * z * (1.0f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
     if (kind == kSquaredRelu) return z > 0.0f ? z * z : 0.0f;
     if (kind == kRelu) return fmaxf(z, 0.0f);
+    if (kind == kTanh) return tanhf(z);
     return z / (1.0f + expf(-z));
+}
+
+// What a gated linear unit makes of a gate and an up value: activate(g) * u, or with kClampedSilu the clamped form
+// g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).
+constexpr int kClampedSilu = 6;
+struct GateConstants { float limit, slope, shift; };
+
+__device__ __forceinline__ float gated_value(float g, float u, int kind, const GateConstants& c) {
+    if (kind == kClampedSilu) {
+        g = fminf(g, c.limit);
+        u = fminf(fmaxf(u, -c.limit), c.limit);
+        return g / (1.0f + expf(-c.slope * g)) * (u + c.shift);
+    }
+    return activate(g, kind) * u;
 }
 
 // Programmatic dependent launch. A kernel launched through launch_chained() may start while its

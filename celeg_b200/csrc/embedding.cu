@@ -8,7 +8,8 @@
 namespace celeg_b200 {
 
 // next_w != null: the first half of a split RMSNorm (gemv_bf16.cu) for the norm that follows:
-// xw_out[t, :] = bf16(residual * next_w) and sumsq_out[t] = sum(residual^2).
+// xw_out[t, :] = bf16(residual * next_w) and sumsq_out[t] = sum(residual^2). next_w == null with xw_out given: xw_out is a
+// plain bfloat16 copy of the row, for a first block that reads the stream itself.
 template <typename W>
 __global__ void embedding_kernel(const W* __restrict__ table, const int* tokens, const int* positions,
                                  const float* __restrict__ frequencies,
@@ -31,10 +32,8 @@ __global__ void embedding_kernel(const W* __restrict__ table, const int* tokens,
             v += (i & 1) ? cosf(angle) : sinf(angle);
         }
         dst[i] = v;
-        if (next_w) {
-            xw_out[(size_t)row * hidden + i] = __float2bfloat16_rn(v * next_w[i]);
-            squares += v * v;
-        }
+        if (xw_out) xw_out[(size_t)row * hidden + i] = __float2bfloat16_rn(next_w ? v * next_w[i] : v);
+        if (next_w) squares += v * v;
     }
     if (next_w) {
         squares = block_sum(squares, scratch);
@@ -80,6 +79,13 @@ CELEG_API int celeg_embedding_split_norm(const void* table, int table_dtype, con
                                          float* sumsq_out, int sumsq_stride, cudaStream_t stream) {
     return embedding_checked(table, table_dtype, tokens, nullptr, nullptr, out, rows, hidden, vocab, multiplier, next_w,
                              xw_out, sumsq_out, sumsq_stride, stream);
+}
+
+// The gather and a bfloat16 copy of the rows.
+CELEG_API int celeg_embedding_copy(const void* table, int table_dtype, const int* tokens, float* out, int rows, int hidden,
+                                   int vocab, float multiplier, void* copy, cudaStream_t stream) {
+    return embedding_checked(table, table_dtype, tokens, nullptr, nullptr, out, rows, hidden, vocab, multiplier, nullptr,
+                             copy, nullptr, 0, stream);
 }
 
 // The gather plus the sinusoidal vector of each token's position (frequencies: float32 [(hidden + 1) / 2]); next_w

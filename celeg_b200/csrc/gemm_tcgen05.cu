@@ -34,12 +34,13 @@ struct TcGemmParams {
     void* c;
     int ldc;
     int* error_flag;
-    int activation;        // kTcActivation: which (common.cuh)
+    int activation;        // kTcActivation: which (common.cuh); kTcSwiGlu: of the gate, or kClampedSilu with its constants
     // Grouped product (null: plain): B holds one [group_rows, k] matrix per group, one after the other, and the
     // device-made table (int32: [0] tiles, then from [4] on (group, first row of A and C, rows) per tile) says which
     // rows of A meet which group; blockIdx.y is the tile, blocks beyond the table's count leave at once.
     const int* table;
     int group_rows;
+    GateConstants gate;
 };
 
 template <int BN, int STAGES, int EPI>
@@ -97,8 +98,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             const unsigned b_dst = a_dst + kBytesA;
             tma_load_2d(a_dst, &map_a, bar, kt * kTileK, m0);
             if (EPI == kTcSwiGlu) {
-                tma_load_2d(b_dst, &map_b, bar, kt * kTileK, n0);                      // gate rows
-                tma_load_2d(b_dst + kBytesB / 2, &map_b, bar, kt * kTileK, p.n + n0);  // their up rows
+                tma_load_2d(b_dst, &map_b, bar, kt * kTileK, b_row0);                       // gate rows
+                tma_load_2d(b_dst + kBytesB / 2, &map_b, bar, kt * kTileK, p.n + b_row0);   // their up rows
             } else {
                 tma_load_2d(b_dst, &map_b, bar, kt * kTileK, b_row0);
             }
@@ -157,7 +158,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     for (int i = 0; i < 32; ++i) {
                         const float g = __bfloat162float(__float2bfloat16_rn(v[i]));
                         const float up = __bfloat162float(__float2bfloat16_rn(u[i]));
-                        v[i] = activate(g, p.activation) * up;
+                        v[i] = gated_value(g, up, p.activation, p.gate);
                     }
                 }
             }
@@ -298,8 +299,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                     const unsigned b_dst = a_dst + kBytesA;
                     tma_load_2d(a_dst, &map_a, bar, kt * kTileK, m0);
                     if (EPI == kTcSwiGlu) {
-                        tma_load_2d(b_dst, &map_b, bar, kt * kTileK, n0);
-                        tma_load_2d(b_dst + kBytesB / 2, &map_b, bar, kt * kTileK, p.n + n0);
+                        tma_load_2d(b_dst, &map_b, bar, kt * kTileK, b_row0);
+                        tma_load_2d(b_dst + kBytesB / 2, &map_b, bar, kt * kTileK, p.n + b_row0);
                     } else {
                         tma_load_2d(b_dst, &map_b, bar, kt * kTileK, b_row0);
                     }
@@ -381,7 +382,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                         for (int i = 0; i < 32; ++i) {
                             const float g = __bfloat162float(__float2bfloat16_rn(v[i]));
                             const float up = __bfloat162float(__float2bfloat16_rn(u[i]));
-                            v[i] = activate(g, p.activation) * up;
+                            v[i] = gated_value(g, up, p.activation, p.gate);
                         }
                     }
                 }
@@ -556,7 +557,8 @@ static int launch_grouped(const CUtensorMap& map_a, const CUtensorMap& map_b, co
         set_error("gemm_tcgen05_grouped: %s", cudaGetErrorString(status));
         return -2;
     }
-    dim3 grid((p.n + BN - 1) / BN, max_tiles);
+    constexpr int out_columns = EPI == kTcSwiGlu ? BN / 2 : BN;
+    dim3 grid((p.n + out_columns - 1) / out_columns, max_tiles);
     kernel<<<grid, kGemmThreads, smem, stream>>>(map_a, map_b, p);
     return check_launch("gemm_tcgen05_grouped");
 }
@@ -597,7 +599,7 @@ CELEG_API int celeg_gemm_tcgen05(const void* a, int lda, const void* b, int ldb,
     if (!tensor_map_for(b, b_rows, k, ldb, epilogue == kTcSwiGlu ? bn / 2 : bn, &map_b)) return -3;
     TcGemmParams p{m, n, k, c, ldc, error_flag,
                    epilogue >= kTcActivation ? epilogue - kTcActivation : (epilogue == kTcSwiGlu ? gate_activation : 0),
-                   nullptr, 0};
+                   nullptr, 0, {0.0f, 0.0f, 0.0f}};
     if (epilogue > kTcActivation) epilogue = kTcActivation;
 #define CELEG_TC_DISPATCH(BN, STAGES)                                                        \
     switch (epilogue) {                                                                      \
@@ -635,35 +637,41 @@ CELEG_API int celeg_gemm_tcgen05(const void* a, int lda, const void* b, int ldb,
 // Grouped product: c[r, :n] = a[r, :k] * b[g(r)][:n, :k]^T, where b holds `groups` matrices of n rows one after the
 // other and the device-made table (see TcGemmParams) assigns runs of rows of a to groups in tiles of at most 128
 // rows. max_tiles bounds the table's tiles and sizes the grid; rows of a: a_rows. epilogue 0 (bfloat16) or 3.. (an
-// activation). The same kernel as the plain product's one-tile-a-block forms; wide_tiles: -1 = chosen from n, 0 / 1.
+// activation), or 16 + kind: every group has n gate rows, then n up rows, and c [rows, n] is what gated_value() makes of the
+// two products (limit, slope, shift: its constants). The same kernel as the plain product's one-tile-a-block forms;
+// wide_tiles: -1 = chosen from n, 0 / 1.
 CELEG_API int celeg_gemm_tcgen05_grouped(const void* a, int lda, int a_rows, const void* b, int ldb, int groups, void* c,
                                          int ldc, const int* table, int max_tiles, int n, int k, int epilogue,
-                                         int* error_flag, int wide_tiles, cudaStream_t stream) {
+                                         float limit, float slope, float shift, int* error_flag, int wide_tiles,
+                                         cudaStream_t stream) {
     CELEG_REQUIRE(a_rows > 0 && n > 0 && k > 0 && groups > 0 && max_tiles >= 0 && table != nullptr,
                   "gemm_tcgen05_grouped: invalid sizes rows=%d n=%d k=%d groups=%d tiles=%d", a_rows, n, k, groups, max_tiles);
     CELEG_REQUIRE(k % 8 == 0 && lda % 8 == 0 && ldb % 8 == 0 && lda >= k && ldb >= k,
                   "gemm_tcgen05_grouped: k=%d, lda=%d and ldb=%d must be multiples of 8 and cover k", k, lda, ldb);
     CELEG_REQUIRE((((size_t)a | (size_t)b) & 15) == 0, "gemm_tcgen05_grouped: operands must be 16-byte aligned");
     CELEG_REQUIRE(ldc >= n && error_flag != nullptr, "gemm_tcgen05_grouped: ldc=%d is smaller than n=%d, or no error flag", ldc, n);
-    CELEG_REQUIRE(epilogue == kTcStoreBf16 || (epilogue >= kTcActivation && epilogue <= 6),
+    const bool gated = epilogue >= 16 && epilogue <= 16 + kClampedSilu;
+    CELEG_REQUIRE(gated || epilogue == kTcStoreBf16 || (epilogue >= kTcActivation && epilogue <= kTcActivation + kSquaredRelu),
                   "gemm_tcgen05_grouped: unknown epilogue %d", epilogue);
     CELEG_REQUIRE(max_tiles <= 65535, "gemm_tcgen05_grouped: %d tiles exceed one launch", max_tiles);
     if (max_tiles == 0) return 0;
     // wide outputs: tiles of 128 x 256 (half as many passes over the rows); else 128 x 128, two blocks per SM
-    const bool wide = wide_tiles < 0 ? n >= 1024 : wide_tiles != 0;
+    const int b_rows = gated ? 2 * n : n;          // of a group
+    bool wide = wide_tiles < 0 ? b_rows >= 1024 : wide_tiles != 0;
+    // many tiles: the persistent form (128 x 256 tiles, two accumulators, the epilogue under the next tile's MMAs)
+    const bool persistent = wide_tiles < 0 && max_tiles * ((b_rows + 255) / 256) >= 148;
+    wide = wide || persistent;
     CUtensorMap map_a, map_b;
     if (!tensor_map_for(a, a_rows, k, lda, kTileM, &map_a)) return -3;
-    if (!tensor_map_for(b, (long long)groups * n, k, ldb, wide ? 256 : 128, &map_b)) return -3;
-    TcGemmParams p{a_rows, n, k, c, ldc, error_flag, epilogue >= kTcActivation ? epilogue - kTcActivation : 0, table, n};
-    const bool store = epilogue == kTcStoreBf16;
-    if (wide_tiles < 0 && max_tiles * ((n + 255) / 256) >= 148) {
-        // many tiles: the persistent form (128 x 256 tiles, two accumulators, the epilogue under the next tile's MMAs)
-        if (!tensor_map_for(b, (long long)groups * n, k, ldb, 256, &map_b)) return -3;
-        return store ? launch_tc_persistent<kTcStoreBf16>(map_a, map_b, p, stream, max_tiles)
-                     : launch_tc_persistent<kTcActivation>(map_a, map_b, p, stream, max_tiles);
-    }
-    if (wide) return store ? launch_grouped<256, 4, kTcStoreBf16>(map_a, map_b, p, max_tiles, stream)
-                           : launch_grouped<256, 4, kTcActivation>(map_a, map_b, p, max_tiles, stream);
-    return store ? launch_grouped<128, 3, kTcStoreBf16>(map_a, map_b, p, max_tiles, stream)
-                 : launch_grouped<128, 3, kTcActivation>(map_a, map_b, p, max_tiles, stream);
+    if (!tensor_map_for(b, (long long)groups * b_rows, k, ldb, (wide ? 256 : 128) / (gated ? 2 : 1), &map_b)) return -3;
+    TcGemmParams p{a_rows, n, k, c, ldc, error_flag,
+                   gated ? epilogue - 16 : epilogue >= kTcActivation ? epilogue - kTcActivation : 0, table, b_rows,
+                   {limit, slope, shift}};
+#define CELEG_TC_GROUPED(EPI)                                                                        \
+    (persistent ? launch_tc_persistent<EPI>(map_a, map_b, p, stream, max_tiles)                      \
+     : wide     ? launch_grouped<256, 4, EPI>(map_a, map_b, p, max_tiles, stream)                    \
+                : launch_grouped<128, 3, EPI>(map_a, map_b, p, max_tiles, stream))
+    if (gated) return CELEG_TC_GROUPED(kTcSwiGlu);
+    return epilogue == kTcStoreBf16 ? CELEG_TC_GROUPED(kTcStoreBf16) : CELEG_TC_GROUPED(kTcActivation);
+#undef CELEG_TC_GROUPED
 }

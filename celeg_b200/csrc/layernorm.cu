@@ -11,7 +11,8 @@
 //
 //   rmsnorm_strided   y[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w over `width` columns of rows that lie `stride`
 //                     elements apart (a slice of a fused projection's result)
-//   sigmoid_gate      values[t, c] *= sigmoid(gate[t, c]) in place, gate float32 or of the activation type
+//   sigmoid_gate      values[t, c] *= sigmoid(gate[t, c / per]) in place, gate float32 or of the activation type, one
+//                     gate for `per` neighbouring columns (1: one a column; a head's size: one a head)
 #include "common.cuh"
 
 namespace celeg_b200 {
@@ -185,13 +186,13 @@ __global__ void rmsnorm_strided_kernel(const A* in, long long in_stride, const f
 
 template <typename A, typename G>
 __global__ void sigmoid_gate_kernel(A* values, long long stride, const G* gate, long long gate_stride, int tokens,
-                                    int width) {
+                                    int width, int per) {
     chain_release();
     chain_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)tokens * width) return;
     const int t = (int)(i / width), c = (int)(i % width);
-    const float g = 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + c])));
+    const float g = 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + c / per])));
     A* cell = values + (size_t)t * stride + c;
     *cell = from_float<A>(to_float(*cell) * g);
 }
@@ -199,7 +200,7 @@ __global__ void sigmoid_gate_kernel(A* values, long long stride, const G* gate, 
 // four neighbours a thread (rows whose widths and strides are multiples of four, 16-byte aligned gate rows)
 template <typename A, typename G>
 __global__ void sigmoid_gate_vec4_kernel(A* values, long long stride, const G* gate, long long gate_stride, int tokens,
-                                         int width) {
+                                         int width, int per) {
     chain_release();
     chain_wait();
     const int quads = width >> 2;
@@ -207,12 +208,12 @@ __global__ void sigmoid_gate_vec4_kernel(A* values, long long stride, const G* g
     if (i >= (long long)tokens * quads) return;
     const int t = (int)(i / quads), c = 4 * (int)(i % quads);
     A* cell = values + (size_t)t * stride + c;
-    const G* g = gate + (size_t)t * gate_stride + c;
+    const G* g = gate + (size_t)t * gate_stride + c / per;      // (per: 1, or a multiple of four)
     float v[4], z[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
         v[e] = to_float(cell[e]);
-        z[e] = to_float(g[e]);
+        z[e] = to_float(g[per == 1 ? e : 0]);
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) cell[e] = from_float<A>(v[e] / (1.0f + __expf(-z[e])));
@@ -280,29 +281,29 @@ CELEG_API int celeg_rmsnorm_strided(const void* in, long long in_stride, const f
     return check_launch("rmsnorm_strided");
 }
 
-// gate_dtype: the type of `gate` (float32 sums of a product, or the activation type)
+// gate_dtype: the type of `gate` (float32 sums of a product, or the activation type); per: columns that share a gate
 CELEG_API int celeg_sigmoid_gate(void* values, long long stride, const void* gate, long long gate_stride, int tokens,
-                                 int width, int act_dtype, int gate_dtype, cudaStream_t stream) {
-    CELEG_REQUIRE(tokens >= 0 && width > 0 && stride >= width && gate_stride >= width,
+                                 int width, int per, int act_dtype, int gate_dtype, cudaStream_t stream) {
+    CELEG_REQUIRE(tokens >= 0 && width > 0 && per > 0 && width % per == 0 && stride >= width && gate_stride >= width / per,
                   "sigmoid_gate: invalid sizes tokens=%d width=%d strides %lld / %lld", tokens, width, stride, gate_stride);
     CELEG_REQUIRE((act_dtype == kFloat32 || act_dtype == kBFloat16) && (gate_dtype == kFloat32 || gate_dtype == act_dtype),
                   "sigmoid_gate: dtype codes %d / %d", act_dtype, gate_dtype);
     if (tokens == 0) return 0;
-    if (act_dtype == kBFloat16 && gate_dtype == kFloat32 && width % 4 == 0 && stride % 4 == 0 && gate_stride % 4 == 0) {
+    if (act_dtype == kBFloat16 && gate_dtype == kFloat32 && width % 4 == 0 && stride % 4 == 0 && (per == 1 || per % 4 == 0)) {
         const unsigned quad_blocks = (unsigned)(((long long)tokens * (width / 4) + 255) / 256);
         launch_chained(sigmoid_gate_vec4_kernel<__nv_bfloat16, float>, quad_blocks, 256, 0, stream, (__nv_bfloat16*)values,
-                       stride, (const float*)gate, gate_stride, tokens, width);
+                       stride, (const float*)gate, gate_stride, tokens, width, per);
         return check_launch("sigmoid_gate");
     }
     const unsigned blocks = (unsigned)(((long long)tokens * width + 255) / 256);
     if (act_dtype == kFloat32)
         launch_chained(sigmoid_gate_kernel<float, float>, blocks, 256, 0, stream, (float*)values, stride,
-                       (const float*)gate, gate_stride, tokens, width);
+                       (const float*)gate, gate_stride, tokens, width, per);
     else if (gate_dtype == kFloat32)
         launch_chained(sigmoid_gate_kernel<__nv_bfloat16, float>, blocks, 256, 0, stream, (__nv_bfloat16*)values, stride,
-                       (const float*)gate, gate_stride, tokens, width);
+                       (const float*)gate, gate_stride, tokens, width, per);
     else
         launch_chained(sigmoid_gate_kernel<__nv_bfloat16, __nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)values,
-                       stride, (const __nv_bfloat16*)gate, gate_stride, tokens, width);
+                       stride, (const __nv_bfloat16*)gate, gate_stride, tokens, width, per);
     return check_launch("sigmoid_gate");
 }

@@ -4,7 +4,8 @@
 //   route      from z = W_r h (a product with float32 sums, made before): s = softmax(z) over all experts; the `top`
 //              experts with the largest s + correction are chosen (ties: the lower index), their weights are
 //              s / (sum of the chosen s + 1e-20); also the sigmoid of one more column of z, the gate of a shared
-//              expert. One warp a token.
+//              expert. One warp a token. Or s = sigmoid(z) element by element, and weights that are the chosen s as
+//              they are.
 //   group      pairs (token, choice) ordered by expert: the source row of every place, the place of every pair,
 //              and a table of row tiles (expert, first place, rows) for the products. One block, one launch;
 //              the order inside an expert is not fixed, and no result depends on it.
@@ -14,7 +15,8 @@
 //              The grid is sized for the most tiles the step can have; blocks beyond the table leave at once,
 //              so nothing about the launch depends on the routing (CUDA graphs replay it).
 //   few pairs  out[pair] = act(x[token(pair)] . W_e^T) with a warp per output element row: the weights of the
-//              chosen experts stream once, no grouping.
+//              chosen experts stream once, no grouping. Gated experts (matrices [gate rows | up rows]): the warp forms both
+//              sums of an inner column and writes what the gate makes of them.
 //   combine    y[t] = sum_k weight[t, k] out[place(t, k)] (+ gate[t] shared[t]), summed in the order of k.
 #include <mma.h>
 
@@ -33,7 +35,8 @@ __device__ __forceinline__ float expert_activation(float z, int kind) {
 // logits: float32 [tokens, stride] = h W_r^T from a product with float32 sums (column `experts`, if asked for, is the
 // shared expert's gate before its sigmoid). One warp a token: softmax over all experts, the choice, the weights.
 __global__ void moe_route_kernel(const float* logits, int stride, const float* bias, const float* correction, int gate_column,
-                                 int* chosen, float* weights, float* shared_gate, int tokens, int experts, int top) {
+                                 int* chosen, float* weights, float* shared_gate, int tokens, int experts, int top,
+                                 int sigmoid_scores, int renormalize) {
     extern __shared__ float route_smem[];          // per warp: scores [experts]
     chain_release();
     chain_wait();
@@ -43,20 +46,26 @@ __global__ void moe_route_kernel(const float* logits, int stride, const float* b
     float* scores = route_smem + (size_t)warp * experts;
     const float* row = logits + (size_t)t * stride;
     if (gate_column >= 0 && lane == 0) shared_gate[t] = 1.0f / (1.0f + expf(-row[gate_column]));
-    float largest = -INFINITY;
     // (a bias of the logits shifts choice and weights alike)
-    for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, row[e] + (bias ? bias[e] : 0.0f));
-    largest = warp_max(largest);
-    float total = 0.0f;
-    for (int e = lane; e < experts; e += 32) {
-        const float p = expf(row[e] + (bias ? bias[e] : 0.0f) - largest);
-        scores[e] = p;
-        total += p;
+    if (sigmoid_scores) {
+        for (int e = lane; e < experts; e += 32)
+            scores[e] = 1.0f / (1.0f + expf(-(row[e] + (bias ? bias[e] : 0.0f))));
+        __syncwarp();
+    } else {
+        float largest = -INFINITY;
+        for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, row[e] + (bias ? bias[e] : 0.0f));
+        largest = warp_max(largest);
+        float total = 0.0f;
+        for (int e = lane; e < experts; e += 32) {
+            const float p = expf(row[e] + (bias ? bias[e] : 0.0f) - largest);
+            scores[e] = p;
+            total += p;
+        }
+        total = warp_sum(total);
+        __syncwarp();
+        for (int e = lane; e < experts; e += 32) scores[e] = scores[e] / total;
+        __syncwarp();
     }
-    total = warp_sum(total);
-    __syncwarp();
-    for (int e = lane; e < experts; e += 32) scores[e] = scores[e] / total;
-    __syncwarp();
     // the `top` largest of s + correction, one after the other; a taken expert is marked by a negative score
     // (scores are not negative)
     float picked_sum = 0.0f;
@@ -86,6 +95,7 @@ __global__ void moe_route_kernel(const float* logits, int stride, const float* b
         }
         __syncwarp();
     }
+    if (!renormalize) return;
     const float inv = 1.0f / (picked_sum + 1e-20f);
     for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= inv;
 }
@@ -278,18 +288,9 @@ __global__ void __launch_bounds__(128) expert_product_mma_kernel(const ExpertPro
 
 // Few pairs: one warp per (pair, output element); the experts' matrices stream once each (pairs that chose the same
 // expert meet in the L2).
+// One warp's sum of row . w over k.
 template <typename A>
-__global__ void expert_rows_kernel(const A* x, int x_stride, int pairs_per_row, const int* chosen, const A* weights,
-                                   long long expert_stride, int w_stride, A* out, int out_stride, int pairs, int n, int k,
-                                   int activation, int vectors) {
-    chain_release();
-    chain_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-    const int j = blockIdx.x * warps + warp;
-    const int pair = blockIdx.y;
-    if (j >= n) return;
-    const A* row = x + (size_t)(pair / pairs_per_row) * x_stride;
-    const A* w = weights + (size_t)chosen[pair] * expert_stride + (size_t)j * w_stride;
+__device__ __forceinline__ float expert_row_sum(const A* row, const A* w, int k, int lane, int vectors) {
     float sum = 0.0f;
     if (sizeof(A) == 2 && vectors) {
         // 8 elements a load, four loads of the weights in flight a lane
@@ -319,8 +320,29 @@ __global__ void expert_rows_kernel(const A* x, int x_stride, int pairs_per_row, 
     } else {
         for (int c = lane; c < k; c += 32) sum = fmaf(to_float(row[c]), to_float(w[c]), sum);
     }
-    sum = warp_sum(sum);
-    if (lane == 0) out[(size_t)pair * out_stride + j] = from_float<A>(expert_activation(sum, activation));
+    return warp_sum(sum);
+}
+
+// n: output columns; GATED: the experts' matrices have 2 n rows (n gate rows, then n up rows)
+template <typename A, bool GATED>
+__global__ void expert_rows_kernel(const A* x, int x_stride, int pairs_per_row, const int* chosen, const A* weights,
+                                   long long expert_stride, int w_stride, A* out, int out_stride, int pairs, int n, int k,
+                                   int activation, int vectors, const GateConstants constants) {
+    chain_release();
+    chain_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int j = blockIdx.x * warps + warp;
+    const int pair = blockIdx.y;
+    if (j >= n) return;
+    const A* row = x + (size_t)(pair / pairs_per_row) * x_stride;
+    const A* w = weights + (size_t)chosen[pair] * expert_stride + (size_t)j * w_stride;
+    const float sum = expert_row_sum<A>(row, w, k, lane, vectors);
+    if (GATED) {
+        const float up = expert_row_sum<A>(row, w + (size_t)n * w_stride, k, lane, vectors);
+        if (lane == 0) out[(size_t)pair * out_stride + j] = from_float<A>(gated_value(sum, up, activation, constants));
+    } else if (lane == 0) {
+        out[(size_t)pair * out_stride + j] = from_float<A>(expert_activation(sum, activation));
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ combine
@@ -380,7 +402,8 @@ __global__ void moe_combine_vec_kernel(const __nv_bfloat16* expert_out, int out_
 using namespace celeg_b200;
 
 CELEG_API int celeg_moe_route(const float* logits, int stride, const float* bias, const float* correction, int gate_column, int* chosen,
-                              float* weights, float* shared_gate, int tokens, int experts, int top, cudaStream_t stream) {
+                              float* weights, float* shared_gate, int tokens, int experts, int top, int sigmoid_scores,
+                              int renormalize, cudaStream_t stream) {
     CELEG_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && stride >= experts,
                   "moe_route: invalid sizes tokens=%d experts=%d top=%d stride=%d", tokens, experts, top, stride);
     CELEG_REQUIRE(experts <= 2048, "moe_route: %d experts exceed a block's shared memory", experts);
@@ -391,7 +414,7 @@ CELEG_API int celeg_moe_route(const float* logits, int stride, const float* bias
     const size_t smem = (size_t)warps * experts * sizeof(float);
     const unsigned blocks = (unsigned)((tokens + warps - 1) / warps);
     launch_chained(moe_route_kernel, blocks, warps * 32, smem, stream, logits, stride, bias, correction, gate_column, chosen,
-                   weights, shared_gate, tokens, experts, top);
+                   weights, shared_gate, tokens, experts, top, sigmoid_scores, renormalize);
     return check_launch("moe_route");
 }
 
@@ -446,11 +469,14 @@ CELEG_API int celeg_expert_product(const void* x, int x_stride, const int* sourc
     return check_launch("expert_product");
 }
 
-// out[pair, :n] = act(x[pair / pairs_per_row] . W[chosen[pair]]^T), for few pairs
+// out[pair, :n] = act(x[pair / pairs_per_row] . W[chosen[pair]]^T), for few pairs; gated: W has n gate rows, then n up
+// rows, and out is what gated_value() makes of the two sums
 CELEG_API int celeg_expert_rows(const void* x, int x_stride, int pairs_per_row, const int* chosen, const void* weights,
                                 long long expert_stride, int w_stride, void* out, int out_stride, int pairs, int n, int k,
-                                int activation, int act_dtype, cudaStream_t stream) {
-    CELEG_REQUIRE(pairs >= 0 && pairs <= 65535 && n > 0 && k > 0 && pairs_per_row > 0 && activation >= -1 && activation <= 3,
+                                int activation, int gated, float limit, float slope, float shift, int act_dtype,
+                                cudaStream_t stream) {
+    CELEG_REQUIRE(pairs >= 0 && pairs <= 65535 && n > 0 && k > 0 && pairs_per_row > 0 &&
+                  (gated ? activation >= 0 && activation <= kClampedSilu : activation >= -1 && activation <= kRelu),
                   "expert_rows: invalid sizes pairs=%d n=%d k=%d activation=%d", pairs, n, k, activation);
     CELEG_REQUIRE(act_dtype == kFloat32 || act_dtype == kBFloat16, "expert_rows: unknown dtype code %d", act_dtype);
     if (pairs == 0) return 0;
@@ -458,14 +484,17 @@ CELEG_API int celeg_expert_rows(const void* x, int x_stride, int pairs_per_row, 
     dim3 grid((n + warps - 1) / warps, pairs);
     const int vectors = k % 8 == 0 && x_stride % 8 == 0 && w_stride % 8 == 0 && expert_stride % 8 == 0 &&
                         (((size_t)x | (size_t)weights) & 15) == 0;
-    if (act_dtype == kFloat32)
-        launch_chained(expert_rows_kernel<float>, grid, warps * 32, 0, stream, (const float*)x, x_stride, pairs_per_row,
-                       chosen, (const float*)weights, expert_stride, w_stride, (float*)out, out_stride, pairs, n, k,
-                       activation, 0);
-    else
-        launch_chained(expert_rows_kernel<__nv_bfloat16>, grid, warps * 32, 0, stream, (const __nv_bfloat16*)x, x_stride,
-                       pairs_per_row, chosen, (const __nv_bfloat16*)weights, expert_stride, w_stride, (__nv_bfloat16*)out,
-                       out_stride, pairs, n, k, activation, vectors);
+    const GateConstants constants = {limit, slope, shift};
+#define CELEG_EXPERT_ROWS(A, GATED)                                                                                       \
+    launch_chained(expert_rows_kernel<A, GATED>, grid, warps * 32, 0, stream, (const A*)x, x_stride, pairs_per_row, chosen, \
+                   (const A*)weights, expert_stride, w_stride, (A*)out, out_stride, pairs, n, k, activation,              \
+                   sizeof(A) == 2 ? vectors : 0, constants)
+    if (act_dtype == kFloat32) {
+        if (gated) CELEG_EXPERT_ROWS(float, true); else CELEG_EXPERT_ROWS(float, false);
+    } else {
+        if (gated) CELEG_EXPERT_ROWS(__nv_bfloat16, true); else CELEG_EXPERT_ROWS(__nv_bfloat16, false);
+    }
+#undef CELEG_EXPERT_ROWS
     return check_launch("expert_rows");
 }
 

@@ -196,6 +196,7 @@ class Model:
         if firsts and firsts[0] is not None and rt.small_batch(step.tokens):
             halves = stream.split(firsts[0], 1)
             first = (firsts[0], halves) if halves is not None else None
+        stream.wants_rows = bool(blocks) and getattr(blocks[0], "reads_stream", False)
         self.input.run(stream, step, first)
         for position, entry in enumerate(self.order):
             layer = self.layers[entry.layer]

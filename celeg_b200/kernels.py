@@ -47,7 +47,8 @@ _SIGNATURES = {
     "celeg_attention_generic": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int,
                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                 c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
-    "celeg_qkv_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_float, c_int, c_int,
+    "celeg_qkv_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_float, c_void_p, c_int,
+                          c_int, c_float, c_float, c_int, c_int,
                           c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                           c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                           c_void_p, c_int, c_void_p],
@@ -55,7 +56,17 @@ _SIGNATURES = {
                             c_int, c_void_p],
     "celeg_rmsnorm_strided": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_int,
                               c_void_p],
-    "celeg_sigmoid_gate": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_sigmoid_gate": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_output_norm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float,
+                          c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "celeg_embedding_copy": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+    "celeg_activation_cast": [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_general_delta_scan": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float,
+                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong,
+                                 c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_general_delta_decode": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
+                                   c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int,
+                                   c_void_p, c_int, c_void_p],
     "celeg_bias_store_kv": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_void_p, c_int, c_void_p],
@@ -71,7 +82,7 @@ _SIGNATURES = {
     "celeg_retention_decode_raw": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_int,
                                    c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
     "celeg_activation_columns": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
-    "celeg_glu": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_glu": [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "celeg_scaled_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "celeg_attention_decode": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
@@ -143,15 +154,16 @@ _SIGNATURES = {
     "celeg_head_project": [c_void_p, c_int, c_int, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_int, c_int,
                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "celeg_head_gate": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "celeg_moe_route": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "celeg_moe_route": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                        c_void_p],
     "celeg_moe_group": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "celeg_moe_gather_rows": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "celeg_gemm_tcgen05_grouped": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int,
-                                   c_int, c_int, c_void_p, c_int, c_void_p],
+                                   c_int, c_int, c_float, c_float, c_float, c_void_p, c_int, c_void_p],
     "celeg_expert_product": [c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int,
                              c_int, c_int, c_int, c_int, c_void_p],
     "celeg_expert_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int,
-                          c_int, c_int, c_int, c_void_p],
+                          c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "celeg_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p],
 }
@@ -220,8 +232,9 @@ class SplitNorm:
 
 def embedding(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, multiplier: float = 1.0,
               prepare: Optional[SplitNorm] = None, next_weight: Optional[torch.Tensor] = None,
-              positions: Optional[torch.Tensor] = None, frequencies: Optional[torch.Tensor] = None) -> None:
-    """out[t] = multiplier * table[tokens[t]]. With ``prepare``: also the first half of the norm whose
+              positions: Optional[torch.Tensor] = None, frequencies: Optional[torch.Tensor] = None,
+              copy: Optional[torch.Tensor] = None) -> None:
+    """out[t] = multiplier * table[tokens[t]]; ``copy`` (bfloat16 [>= tokens, hidden]) gets the same rows rounded. With ``prepare``: also the first half of the norm whose
     weight is ``next_weight`` (``prepare.xw`` and one sum of squares per row are written). With ``positions`` and
     ``frequencies`` (float32 [(hidden + 1) // 2]): plus a sinusoidal vector of the position, entry 2i
     sin(p f_i), entry 2i + 1 cos(p f_i)."""
@@ -231,6 +244,7 @@ def embedding(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, mult
     vocab, hidden = table.shape
     assert out.shape[0] >= rows and out.shape[1] == hidden
     if frequencies is not None:
+        assert copy is None
         _need(frequencies, torch.float32, "frequencies")
         _need(positions, torch.int32, "positions")
         assert frequencies.numel() >= (hidden + 1) // 2 and positions.numel() >= rows
@@ -242,6 +256,11 @@ def embedding(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, mult
             hidden, vocab, multiplier, _ptr(next_weight) if prepare is not None else None,
             _ptr(prepare.xw) if prepare is not None else None, _ptr(prepare.sumsq) if prepare is not None else None,
             prepare.sumsq.stride(0) if prepare is not None else 0, _stream()))
+        return
+    if copy is not None:
+        assert prepare is None and copy.dtype == torch.bfloat16 and copy.is_contiguous() and copy.shape[1] == hidden
+        _check(library().celeg_embedding_copy(_ptr(table), dtype_code(table.dtype), _ptr(tokens), _ptr(out), rows, hidden,
+                                              vocab, multiplier, _ptr(copy), _stream()))
         return
     if prepare is None:
         _check(library().celeg_embedding(_ptr(table), dtype_code(table.dtype), _ptr(tokens), _ptr(out), rows, hidden,
@@ -268,6 +287,36 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
     _check(library().celeg_add_rmsnorm(_ptr(residual), _ptr(delta), _ptr(weight), _ptr(out), _ptr(rows), n_rows,
                                        width, eps, int(write_residual and rows is None), dtype_code(out.dtype),
                                        _stream()))
+
+
+def output_norm(residual: torch.Tensor, n_rows: int, rows: Optional[torch.Tensor], norm_weight: Optional[torch.Tensor],
+                eps: float, out: Optional[torch.Tensor], *, place: Optional[torch.Tensor] = None,
+                weights: Optional[torch.Tensor] = None, top: int = 1, bias: Optional[torch.Tensor] = None,
+                prepare: Optional[SplitNorm] = None, next_weight: Optional[torch.Tensor] = None) -> None:
+    """residual[t] += rmsnorm(y[t]) * norm_weight with y[t] = rows[t] (+ bias), or with ``weights`` (float32 [n_rows * top])
+    y[t] = sum_k weights[t, k] rows[place[t * top + k]]; then out[t] = residual[t] rounded to the type of ``out``. ``rows``
+    None: the copy alone. With ``prepare`` the first half of the norm that reads the stream next (weight ``next_weight``)
+    is left in ``prepare`` instead of the copy (csrc/output_norm.cu)."""
+    _need(residual, torch.float32, "residual")
+    width = residual.shape[-1]
+    if prepare is not None:
+        assert out is None and prepare.partials == 1 and prepare.xw.stride(0) == width
+        _need(next_weight, torch.float32, "next_weight")
+        out = prepare.xw
+    if out is not None:
+        assert out.is_contiguous() and out.shape[-1] == width
+    for vector in (norm_weight, weights, bias):
+        if vector is not None:
+            _need(vector, torch.float32, "a vector of output_norm")
+    if rows is not None:
+        assert rows.stride(-1) == 1 and rows.shape[-1] == width
+    out_dtype = out.dtype if out is not None else torch.float32
+    _check(library().celeg_output_norm(
+        _ptr(residual), _ptr(rows), dtype_code(rows.dtype) if rows is not None else dtype_code(out_dtype),
+        rows.stride(0) if rows is not None else 0, _ptr(place), _ptr(weights), top, _ptr(bias), _ptr(norm_weight), eps,
+        _ptr(out), dtype_code(out_dtype), _ptr(next_weight) if prepare is not None else None,
+        _ptr(prepare.sumsq) if prepare is not None else None, prepare.sumsq.stride(0) if prepare is not None else 0, n_rows,
+        width, _stream()))
 
 
 def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, n_rows: int) -> None:
@@ -357,31 +406,38 @@ def _distance_bias(table: Optional[torch.Tensor], q_heads: int) -> Tuple[Optiona
 
 
 def qkv_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_out: torch.Tensor, positions: torch.Tensor,
-                token_span: torch.Tensor, block_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
-                tokens: int, q_heads: int, kv_heads: int, head_dim: int, value_dim: int, key_store: int,
-                value_store: int, page_tokens: int, error_flag: torch.Tensor, *,
+                token_span: torch.Tensor, block_table: torch.Tensor, k_cache: Optional[torch.Tensor],
+                v_cache: Optional[torch.Tensor], tokens: int, q_heads: int, kv_heads: int, head_dim: int, value_dim: int,
+                key_store: int, value_store: int, page_tokens: int, error_flag: torch.Tensor, *,
                 q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
-                frequencies: Optional[torch.Tensor] = None, rotary_dim: int = 0,
+                norm_per_head: bool = False, unit_values_eps: Optional[float] = None,
+                frequencies: Optional[torch.Tensor] = None, rotary_dim: int = 0, interleaved: bool = False,
+                magnitude: float = 1.0,
                 temperature: Optional[Tuple[float, int]] = None, blend: int = 0, lam: float = 0.0,
                 first_values: Optional[torch.Tensor] = None) -> None:
     """Float32 rows [q heads | k heads | v heads | ...] as projected become queries in ``q_out`` and keys and values
     in the tokens' places of the paged cache (csrc/attention_prepare.cu), after, in this order: the biases; one RMS
     norm over the whole q projection and one over the whole k projection (``q_norm`` / ``k_norm``, as wide as the
-    projections); the rotation of the first ``rotary_dim`` entries of every q and k head in pairs (i, i + half) by
-    position x ``frequencies``; ``temperature`` = (coef, every): q times 1 + coef ln(floor((position + 1) / every) + 1);
+    projections), or with ``norm_per_head`` one a head (weights as wide as a head); the rotation of the first
+    ``rotary_dim`` entries of every q and k head in pairs (i, i + half), or of neighbours with ``interleaved``, by
+    position x ``frequencies``, cosine and sine times ``magnitude``; ``temperature`` = (coef, every): q times 1 + coef ln(floor((position + 1) / every) + 1);
     ``blend`` 1: the values are noted in ``first_values`` (float32 [tokens, kv_heads * value_dim]); 2: v becomes
-    (1 - lam) v + lam first_values. One rounding."""
+    (1 - lam) v + lam first_values; with ``unit_values_eps`` every value head is divided by its root mean square. One
+    rounding. ``kv_heads`` 0 without caches: rows of queries alone."""
     _need(proj, torch.float32, "proj")
     for vector in (bias, q_norm, k_norm, frequencies, first_values):
         if vector is not None:
             _need(vector, torch.float32, "a vector of qkv_prepare")
-    assert q_out.dtype == k_cache.dtype == v_cache.dtype and q_out.stride(-1) == 1 and proj.stride(-1) == 1
+    assert q_out.stride(-1) == 1 and proj.stride(-1) == 1
+    assert kv_heads == 0 or q_out.dtype == k_cache.dtype == v_cache.dtype
     coef, every = temperature if temperature else (0.0, 0)
     _check(library().celeg_qkv_prepare(
-        _ptr(proj), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), norm_eps, _ptr(frequencies), rotary_dim,
-        float(coef), int(every), blend, lam, _ptr(first_values), first_values.stride(0) if first_values is not None else 0,
+        _ptr(proj), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), norm_eps, int(norm_per_head),
+        int(unit_values_eps is not None), float(unit_values_eps or 0.0), _ptr(frequencies), rotary_dim, int(interleaved),
+        magnitude, float(coef), int(every), blend, lam, _ptr(first_values), first_values.stride(0) if first_values is not None else 0,
         _ptr(q_out), q_out.stride(0), _ptr(positions), _ptr(token_span), _ptr(block_table), block_table.stride(0),
-        _ptr(k_cache), _ptr(v_cache), k_cache.stride(0), v_cache.stride(0), tokens, q_heads, kv_heads, head_dim, value_dim,
+        _ptr(k_cache), _ptr(v_cache), k_cache.stride(0) if k_cache is not None else 0,
+        v_cache.stride(0) if v_cache is not None else 0, tokens, q_heads, kv_heads, head_dim, value_dim,
         key_store, value_store, page_tokens, _ptr(error_flag), dtype_code(q_out.dtype), _stream()))
 
 
@@ -409,11 +465,11 @@ def rmsnorm_strided(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, ep
                                            x.shape[-1], eps, dtype_code(x.dtype), _stream()))
 
 
-def sigmoid_gate(values: torch.Tensor, gate: torch.Tensor, tokens: int, width: int) -> None:
-    """values[t, c] *= sigmoid(gate[t, c]) for c < width, in place; ``gate`` float32 or of the values' type."""
+def sigmoid_gate(values: torch.Tensor, gate: torch.Tensor, tokens: int, width: int, per: int = 1) -> None:
+    """values[t, c] *= sigmoid(gate[t, c // per]) for c < width, in place; ``gate`` float32 or of the values' type."""
     assert values.stride(-1) == 1 and gate.stride(-1) == 1
     _check(library().celeg_sigmoid_gate(_ptr(values), values.stride(0), _ptr(gate), gate.stride(0), tokens, width,
-                                        dtype_code(values.dtype), dtype_code(gate.dtype), _stream()))
+                                        per, dtype_code(values.dtype), dtype_code(gate.dtype), _stream()))
 
 
 def bias_store_kv(proj: torch.Tensor, bias: Optional[torch.Tensor], q_out: torch.Tensor, positions: torch.Tensor,
@@ -550,7 +606,9 @@ def attention_prefill_tcgen05(q: torch.Tensor, q_row_stride: int, out: torch.Ten
         head_dim, page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, _ptr(error_flag), _stream()))
 
 
-ACT_GELU_ERF, ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED, ACT_RELU = 0, 1, 2, 3, 4      # codes of csrc/common.cuh: activate()
+ACT_GELU_ERF, ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED, ACT_RELU, ACT_TANH = 0, 1, 2, 3, 4, 5      # codes of csrc/common.cuh: activate()
+GATE_CLAMPED_SILU = 6      # beside them for gated pairs: g' sigmoid(slope g') (u' + shift), g' and u' cut off at a limit
+NO_GATE_CONSTANTS = (0.0, 0.0, 0.0)      # (limit, slope, shift) of GATE_CLAMPED_SILU
 GEMV_MAX_ROWS = 16
 GEMV_STORE, GEMV_STORE_F32, GEMV_ADD_RESIDUAL, GEMV_SWIGLU, GEMV_CONV, GEMV_ACTIVATION = 0, 1, 2, 3, 4, 5
 
@@ -642,9 +700,11 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, tokens: int, inner: int) ->
     _check(library().celeg_swiglu(_ptr(gate_up), _ptr(out), tokens, inner, dtype_code(gate_up.dtype), _stream()))
 
 
-def glu(gate_up: torch.Tensor, out: torch.Tensor, tokens: int, inner: int, kind: int) -> None:
-    """out[:tokens] = act(gate) * up of rows [gate | up] (``inner`` each), ``kind`` one of ACT_*."""
-    _check(library().celeg_glu(_ptr(gate_up), _ptr(out), tokens, inner, kind, dtype_code(gate_up.dtype), _stream()))
+def glu(gate_up: torch.Tensor, out: torch.Tensor, tokens: int, inner: int, kind: int,
+        constants: Tuple[float, float, float] = NO_GATE_CONSTANTS) -> None:
+    """out[:tokens] = act(gate) * up of rows [gate | up] (``inner`` each), ``kind`` one of ACT_*, or GATE_CLAMPED_SILU with
+    its ``constants``."""
+    _check(library().celeg_glu(_ptr(gate_up), _ptr(out), tokens, inner, kind, *constants, dtype_code(gate_up.dtype), _stream()))
 
 
 def gemm_f32(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, accumulate: bool = False) -> None:
@@ -886,6 +946,56 @@ def retention_decode_raw(proj: torch.Tensor, offsets: Tuple[int, int, int], deca
                                                 input_act, _ptr(raw_out), _stream()))
 
 
+# ------------------------------------------------------------------------------- generalised delta rule
+DELTA_CHUNK = 8             # tokens whose sums over the state are formed together (csrc/general_delta.cu)
+
+
+def activation_cast(x: torch.Tensor, out: torch.Tensor, tokens: int, kind: int) -> None:
+    """out[:tokens] = act(x[:tokens]) of float32 columns that lie in wider rows, rounded once to the type of ``out``."""
+    assert x.dtype == torch.float32 and x.stride(-1) == 1 and out.is_contiguous() and x.shape[-1] == out.shape[-1]
+    _check(library().celeg_activation_cast(_ptr(x), x.stride(0), _ptr(out), tokens, out.shape[-1], kind,
+                                           dtype_code(out.dtype), _stream()))
+
+
+def general_delta_scan(proj: torch.Tensor, offsets: Tuple[int, int, int, int], z: torch.Tensor, w0: torch.Tensor,
+                       a_bias: torch.Tensor, unit_eps: float, token_span: torch.Tensor, span_begin: torch.Tensor,
+                       span_slot: torch.Tensor, vectors: torch.Tensor, decay: torch.Tensor, sums: torch.Tensor,
+                       out: torch.Tensor, state: torch.Tensor, slot_stride: int, tokens: int, spans: int, heads: int,
+                       dim: int) -> None:
+    """S <- diag(w) S - b (u^T S) + k v^T, o = S^T r along the step's spans (csrc/general_delta.cu). ``offsets``: columns of
+    (r, k, v, removal rate) in a row of ``proj``; ``z`` [>= tokens, heads * dim] the decay before its bias ``w0``. Scratch,
+    all float32: ``vectors`` tokens * heads * 4 * dim', ``decay`` tokens * heads * dim', ``sums`` heads * tokens * 16
+    elements, dim' = dim rounded up to a multiple of 4."""
+    pad = -(-dim // 4) * 4
+    for tensor in (proj, z, w0, a_bias, vectors, decay, sums, out, state):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert vectors.numel() >= tokens * heads * 4 * pad and decay.numel() >= tokens * heads * pad
+    assert sums.numel() >= heads * tokens * 2 * DELTA_CHUNK and out.is_contiguous() and out.shape[1] == heads * dim
+    _check(library().celeg_general_delta_scan(
+        _ptr(proj), proj.stride(0), *offsets, _ptr(z), z.stride(0), _ptr(w0), _ptr(a_bias), unit_eps, _ptr(token_span),
+        _ptr(span_begin), _ptr(span_slot), _ptr(vectors), _ptr(decay), _ptr(sums), _ptr(out), _ptr(state), slot_stride,
+        tokens, spans, heads, dim, _stream()))
+    global LAUNCHES
+    LAUNCHES += 1          # the vectors, then the scan
+
+
+def general_delta_decode(proj: torch.Tensor, offsets: Tuple[int, int, int, int, int, int], decay_up: torch.Tensor,
+                         w0: torch.Tensor, a_bias: torch.Tensor, norm_weight: torch.Tensor, eps: float, unit_eps: float,
+                         state: torch.Tensor, slot_stride: int, span_slot: torch.Tensor, tokens: int, heads: int, dim: int,
+                         out: torch.Tensor) -> None:
+    """A decoding step of the generalised delta rule between its two projections in one launch: the decay's second product,
+    decay and removal rates, state update, read-out, head norm, weight and sigmoid gate. ``offsets``: columns of (r, k, v,
+    gate, removal rate, the decay's first product) in a row of ``proj`` (float32)."""
+    for tensor in (proj, w0, a_bias, norm_weight, state):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert decay_up.dtype == out.dtype and decay_up.is_contiguous() and decay_up.shape[0] == heads * dim
+    assert out.is_contiguous() and out.shape[1] == heads * dim
+    _check(library().celeg_general_delta_decode(
+        _ptr(proj), proj.stride(0), *offsets, _ptr(decay_up), decay_up.shape[1], _ptr(w0), _ptr(a_bias), _ptr(norm_weight),
+        eps, unit_eps, _ptr(state), slot_stride, _ptr(span_slot), tokens, heads, dim, _ptr(out), dtype_code(out.dtype),
+        _stream()))
+
+
 # ------------------------------------------------------------- gated linear recurrent unit over channels
 def lru_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], taps: torch.Tensor, conv_bias: Optional[torch.Tensor],
                 carried: torch.Tensor, slot_stride: int, token_span: torch.Tensor, span_begin: torch.Tensor,
@@ -1018,12 +1128,14 @@ def moe_max_tiles(pairs: int, experts: int, tile_rows: int = MOE_TILE) -> int:
 
 def moe_route(logits: torch.Tensor, experts: int, correction: Optional[torch.Tensor], gate_column: Optional[int],
               chosen: torch.Tensor, weights: torch.Tensor, shared_gate: Optional[torch.Tensor], tokens: int,
-              top: int, bias: Optional[torch.Tensor] = None) -> None:
+              top: int, bias: Optional[torch.Tensor] = None, sigmoid_scores: bool = False,
+              renormalize: bool = True) -> None:
     """From router logits (float32 [tokens, >= experts], a product with float32 sums; ``bias`` float32 [experts] is
     added to them first): chosen int32 [tokens, top] and weights float32 [tokens, top], the ``top`` experts with the
     largest softmax(logits[:, :experts]) + correction and their softmax scores divided by their sum (without a
     correction that is: the largest logits choose, and the weights are the softmax over the chosen logits alone);
-    shared_gate float32 [tokens] = sigmoid(logits[:, gate_column])."""
+    shared_gate float32 [tokens] = sigmoid(logits[:, gate_column]). ``sigmoid_scores``: the scores are sigmoid(logits)
+    instead of the softmax; ``renormalize`` False: the weights are the chosen scores as they are."""
     _need(chosen, torch.int32, "chosen")
     _need(weights, torch.float32, "weights")
     assert logits.dtype == torch.float32 and logits.stride(-1) == 1 and logits.shape[-1] >= experts
@@ -1032,7 +1144,7 @@ def moe_route(logits: torch.Tensor, experts: int, correction: Optional[torch.Ten
         assert bias.numel() >= experts
     _check(library().celeg_moe_route(_ptr(logits), logits.stride(0), _ptr(bias), _ptr(correction),
                                      -1 if gate_column is None else gate_column, _ptr(chosen), _ptr(weights),
-                                     _ptr(shared_gate), tokens, experts, top, _stream()))
+                                     _ptr(shared_gate), tokens, experts, top, int(sigmoid_scores), int(renormalize), _stream()))
 
 
 def moe_group(chosen: torch.Tensor, tokens: int, experts: int, top: int, place_of_pair: torch.Tensor,
@@ -1060,15 +1172,20 @@ def expert_product_tcgen05_supported(x: torch.Tensor, weights: torch.Tensor) -> 
 
 
 def expert_product_tcgen05(x: torch.Tensor, weights: torch.Tensor, out: torch.Tensor, table: torch.Tensor,
-                           max_tiles: int, activation: int, error_flag: torch.Tensor, wide_tiles: int = -1) -> None:
+                           max_tiles: int, activation: int, error_flag: torch.Tensor, wide_tiles: int = -1,
+                           gated: bool = False, constants: Tuple[float, float, float] = NO_GATE_CONSTANTS) -> None:
     """out[place] = act(x[place] @ weights[expert of the place]^T) on tcgen05 over a tile table of 128-row tiles;
     ``x`` holds the rows in the order of their places. ``activation``: a code of ACT_* or -1. ``wide_tiles``: output
-    tiles of 256 columns (1) or 128 (0); -1: chosen from the shape."""
+    tiles of 256 columns (1) or 128 (0); -1: chosen from the shape. ``gated``: an expert's matrix holds gate rows, then as
+    many up rows, and out [places, half of them] = act(gate) * up (or the clamped form with its ``constants``)."""
     _, n, k = weights.shape
+    if gated:
+        n //= 2
     assert out.dtype == torch.bfloat16 and out.stride(-1) == 1 and out.shape[-1] == n and x.shape[-1] == k
     _check(library().celeg_gemm_tcgen05_grouped(_ptr(x), x.stride(0), x.shape[0], _ptr(weights), weights.stride(1),
                                                 weights.shape[0], _ptr(out), out.stride(0), _ptr(table), max_tiles, n, k,
-                                                TC_STORE if activation < 0 else TC_ACTIVATION + activation,
+                                                TC_GATED + activation if gated else
+                                                TC_STORE if activation < 0 else TC_ACTIVATION + activation, *constants,
                                                 _ptr(error_flag), wide_tiles, _stream()))
 
 
@@ -1084,13 +1201,18 @@ def expert_product(x: torch.Tensor, source: Optional[torch.Tensor], weights: tor
 
 
 def expert_rows(x: torch.Tensor, pairs_per_row: int, chosen: torch.Tensor, weights: torch.Tensor, out: torch.Tensor,
-                pairs: int, activation: int) -> None:
-    """out[pair] = act(x[pair // pairs_per_row] @ weights[chosen[pair]]^T) for few pairs (the weights stream once)."""
+                pairs: int, activation: int, gated: bool = False,
+                constants: Tuple[float, float, float] = NO_GATE_CONSTANTS) -> None:
+    """out[pair] = act(x[pair // pairs_per_row] @ weights[chosen[pair]]^T) for few pairs (the weights stream once).
+    ``gated``: as for :func:`expert_product_tcgen05`."""
     assert x.dtype == weights.dtype == out.dtype and weights.is_contiguous() and x.stride(-1) == 1 and out.stride(-1) == 1
     _, n, k = weights.shape
+    if gated:
+        n //= 2
+    assert out.shape[-1] == n
     _check(library().celeg_expert_rows(_ptr(x), x.stride(0), pairs_per_row, _ptr(chosen), _ptr(weights),
                                        weights.stride(0), weights.stride(1), _ptr(out), out.stride(0), pairs, n, k,
-                                       activation, dtype_code(x.dtype), _stream()))
+                                       activation, int(gated), *constants, dtype_code(x.dtype), _stream()))
 
 
 def moe_combine(expert_out: torch.Tensor, place_of_pair: Optional[torch.Tensor], weights: torch.Tensor,

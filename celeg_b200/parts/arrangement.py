@@ -7,6 +7,8 @@ stream. Interface:
                                      stream.after_layer is the norm that will read the stream after this
                                      layer if its reader takes a split norm (see ResidualStream), else None
     first_norm(step)                 optional: the norm that reads the stream first, under the same condition
+    reads_stream = True              optional: the first thing run() asks for is the stream itself (its rows in the
+                                     activation type), not a norm of it
 
 A part's ``forward(x, out, step)`` gets the normed activations and a buffer for its output; the
 arrangement hands that buffer to the residual stream, which adds it inside the next norm kernel.
@@ -119,3 +121,52 @@ class ParallelResidual:
         stream.add_later_beside(self.delta_b)
         if self.after is not None:
             self.after.run(stream, step)
+
+
+@register_part("arrangement", "output_norm_residual")
+class OutputNormResidual:
+    """x <- x + Norm_1(Mixer(x)); x <- x + Norm_2(FeedForward(x)): the norms act on what the sublayers put out, the
+    sublayers read x itself. One launch a sublayer norms its output, adds it to the float32 stream and leaves x in the
+    activation type for the next one (csrc/output_norm.cu); an output projection's bias (``forward_without_bias``) and the
+    experts' weighted sum (``forward_terms``) are formed in that launch. A part whose last step is a product writes float32
+    rows for it, so the norm's sum sees unrounded outputs."""
+
+    reads_stream = True
+
+    def __init__(self, layer_parts: Mapping, rt: Runtime):
+        self.rt = rt
+        self.mixer_norm = layer_parts["mixer_norm"]
+        self.mixer = layer_parts["mixer"]
+        self.ffn_norm = layer_parts.get("feed_forward_norm")
+        self.ffn = layer_parts.get("feed_forward")
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and (not hasattr(norm, "as_prologue") or norm.as_prologue() is None):
+                raise ValueError("output_norm_residual: the norms must be plain RMS norms")
+        hidden = self.mixer_norm.width
+        self.output = rt.scratch("block.output", hidden, torch.float32)
+        self.delta = rt.scratch("block.delta_a", hidden)
+
+    def _sublayer(self, norm, part, upcoming, stream: ResidualStream, step: StepContext) -> None:
+        x = stream.as_rows(step.tokens)
+        stream.expect(self.output, None, step.tokens)
+        terms = part.forward_terms(x, step) if hasattr(part, "forward_terms") else None
+        if terms is not None:
+            rows, place, weights, top = terms
+            stream.add_normed(norm, step.tokens, rows, place=place, weights=weights, top=top, upcoming=upcoming)
+            return
+        bias = None
+        if hasattr(part, "forward_without_bias"):
+            output = self.output
+            bias = part.forward_without_bias(x, output, step)
+        else:
+            output = self.output if getattr(part, "ends_with_product", False) else self.delta
+            part.forward(x, output, step)
+        stream.add_normed(norm, step.tokens, output, bias=bias, upcoming=upcoming)
+
+    def run(self, stream: ResidualStream, step: StepContext) -> None:
+        after = stream.after_layer
+        if self.ffn is None:
+            self._sublayer(self.mixer_norm, self.mixer, after, stream, step)
+            return
+        self._sublayer(self.mixer_norm, self.mixer, None, stream, step)
+        self._sublayer(self.ffn_norm, self.ffn, after, stream, step)

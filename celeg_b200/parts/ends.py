@@ -6,7 +6,8 @@ names a kind of its own, registered like any other part.
 
 An input part has ``run(stream, step, first)``: write ``stream.residual[:step.tokens]``; ``first`` is
 None or ``(norm weight, SplitNorm)`` of the first block's norm, which the part may prepare (and then sets
-``stream.prepared``). ``vocab_size`` is the number of token ids it takes.
+``stream.prepared``); when ``stream.wants_rows`` it may leave the rows in the activation type in ``stream.rows`` (and then
+sets ``stream.rows_current``). ``vocab_size`` is the number of token ids it takes.
 An output part has ``next_norm(step, n_logits)``: the norm it applies first if it takes it split over the
 last block's closing product and its own (else None), and ``run(stream, step, logit_rows, n_logits,
 logits)``: float32 logits of the stream's rows ``logit_rows[:n_logits]`` (all rows in order when
@@ -55,6 +56,9 @@ class EmbeddingInput:
             kernels.embedding(self.table, tokens, stream.residual, self.multiplier, prepare=split, next_weight=weight,
                               **places)
             stream.prepared = (norm, split)
+        elif stream.wants_rows and stream.rows is not stream.residual and not places:
+            kernels.embedding(self.table, tokens, stream.residual, self.multiplier, copy=stream.rows)
+            stream.rows_current = True
         else:
             kernels.embedding(self.table, tokens, stream.residual, self.multiplier, **places)
 

@@ -17,6 +17,8 @@ from .runtime import Runtime, StepContext
 
 ACTIVATIONS = {"gelu": kernels.ACT_GELU_ERF, "gelu_tanh": kernels.ACT_GELU_TANH, "silu": kernels.ACT_SILU,
                "relu2": kernels.ACT_RELU_SQUARED, "relu": kernels.ACT_RELU}
+# functions of a gate and an up value together, with constants of their own
+GATE_FORMS = {"clamped_silu": kernels.GATE_CLAMPED_SILU}
 
 
 @register_part("feed_forward", "swiglu")
@@ -87,8 +89,11 @@ class MoeFeedForward:
     sigmoid(w_shared_gate . x) when the tensor ``shared_gate`` is given. A tensor ``router_bias`` is added to the
     router's logits. Without a correction the choice falls on the largest logits and the weights are the softmax over
     the chosen logits alone (s_e / sum of the chosen s is that softmax). With ``gated_experts`` an expert is a gated
-    linear unit down_e(act(gate_e(x)) * up_e(x)): gate_e and up_e are stacked into one matrix, the first product
-    leaves [gate | up] rows and an element-wise kernel makes the inner rows.
+    linear unit down_e(act(gate_e(x)) * up_e(x)): gate_e and up_e are stacked into one matrix and the first product
+    writes the inner rows (steps of few tokens and the tcgen05 form; else it leaves [gate | up] rows for an element-wise
+    kernel). ``activation="clamped_silu"`` is then the form g sigmoid(``gate_slope`` g) (u + ``up_shift``) of a gate cut
+    off at ``gate_limit`` and an up value cut off at both signs of it. ``scores="sigmoid"`` takes s = sigmoid(W_router x)
+    in the softmax's place; ``renormalize=False`` leaves the chosen s as the weights.
 
     Steps of few tokens stream the chosen experts' matrices once per (token, choice) pair; larger steps order the
     pairs by expert on the device and run both products tile by tile over a table the device makes, on a grid
@@ -106,9 +111,20 @@ class MoeFeedForward:
         self.experts = int(params["experts"])
         self.top = int(params["top"])
         name = params.get("activation", "relu2")
-        if name not in DenseFeedForward.ACTIVATIONS:
-            raise ValueError(f"moe: unknown activation {name!r}; known: {', '.join(DenseFeedForward.ACTIVATIONS)}")
-        self.activation = DenseFeedForward.ACTIVATIONS[name]
+        self.gated_experts = bool(params.get("gated_experts", False))
+        known = dict(ACTIVATIONS, **GATE_FORMS) if self.gated_experts else ACTIVATIONS
+        if name not in known:
+            raise ValueError(f"moe: unknown activation {name!r}; known: {', '.join(known)}")
+        self.activation = known[name]
+        self.gate_constants = kernels.NO_GATE_CONSTANTS
+        if name == "clamped_silu":
+            self.gate_constants = (float(params["gate_limit"]), float(params.get("gate_slope", 1.0)),
+                                   float(params.get("up_shift", 0.0)))
+        scores = params.get("scores", "softmax")
+        if scores not in ("softmax", "sigmoid"):
+            raise ValueError(f"moe: unknown scores {scores!r}; known: softmax, sigmoid")
+        self.sigmoid_scores = scores == "sigmoid"
+        self.renormalize = bool(params.get("renormalize", True))
         if not 0 < self.top <= self.experts:
             raise ValueError(f"moe: top {self.top} of {self.experts} experts")
         # the router's matrix, with the shared expert's gate as one more row: one product with float32 sums gives both
@@ -118,7 +134,6 @@ class MoeFeedForward:
         self.logits = rt.scratch("moe.logits", int(self.w_router.shape[0]), torch.float32)
         self.correction = rt.vector(weights["correction"]) if "correction" in weights else None
         self.router_bias = rt.vector(weights["router_bias"]) if "router_bias" in weights else None
-        self.gated_experts = bool(params.get("gated_experts", False))
         if self.gated_experts:                                                                        # [E, 2 inner, hidden]
             self.w_up = rt.matrix(torch.stack([torch.cat([weights[f"e{e}.gate"], weights[f"e{e}.up"]], dim=0)
                                                for e in range(self.experts)]))
@@ -142,41 +157,50 @@ class MoeFeedForward:
         self.lowered = rt.flat_scratch("moe.lowered", pairs * self.hidden, rt.act_dtype).view(pairs, self.hidden)
         self.shared_out = rt.scratch("moe.shared_out", self.hidden) if self.shared is not None else None
 
-    def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
+    def _expert_rows(self, x: torch.Tensor, step: StepContext):
+        """Routes and runs both products; returns the row of ``lowered`` for every (token, choice) pair, None when the
+        rows lie in the pairs' own order."""
         t, top = step.tokens, self.top
         pairs = t * top
         gated = self.gated
         self.rt.linear(x, self.w_router, self.logits, t)
         kernels.moe_route(self.logits, self.experts, self.correction, self.experts if gated else None, self.chosen,
-                          self.weights, self.shared_gate if gated else None, t, top, bias=self.router_bias)
+                          self.weights, self.shared_gate if gated else None, t, top, bias=self.router_bias,
+                          sigmoid_scores=self.sigmoid_scores, renormalize=self.renormalize)
         if self.shared is not None:
             self.shared.forward(x, self.shared_out, step)
-        # what the first product writes and which activation its epilogue applies
-        first_out, first_act = (self.paired, -1) if self.gated_experts else (self.raised, self.activation)
+        first = {"gated": self.gated_experts, "constants": self.gate_constants}
         if t <= self.FEW_TOKENS:
-            kernels.expert_rows(x, top, self.chosen, self.w_up, first_out, pairs, first_act)
-            if self.gated_experts:
-                kernels.glu(self.paired, self.raised, pairs, self.inner, self.activation)
+            kernels.expert_rows(x, top, self.chosen, self.w_up, self.raised, pairs, self.activation, **first)
             kernels.expert_rows(self.raised, 1, self.chosen, self.w_down, self.lowered, pairs, -1)
-            place = None
-        elif (self.rt.tensor_core_products != "none" and kernels.expert_product_tcgen05_supported(self.gathered, self.w_up)
-              and kernels.expert_product_tcgen05_supported(self.raised, self.w_down)):
+            return None
+        if (self.rt.tensor_core_products != "none" and kernels.expert_product_tcgen05_supported(self.gathered, self.w_up)
+                and kernels.expert_product_tcgen05_supported(self.raised, self.w_down)):
             kernels.moe_group(self.chosen, t, self.experts, top, self.place, self.source, self.table, tile_rows=128)
             tiles = kernels.moe_max_tiles(pairs, self.experts, 128)
             kernels.moe_gather_rows(x, self.source, self.gathered, pairs)
-            kernels.expert_product_tcgen05(self.gathered, self.w_up, first_out, self.table, tiles, first_act,
-                                           self.rt.error_flag)
-            if self.gated_experts:
-                kernels.glu(self.paired, self.raised, pairs, self.inner, self.activation)
+            kernels.expert_product_tcgen05(self.gathered, self.w_up, self.raised, self.table, tiles, self.activation,
+                                           self.rt.error_flag, **first)
             kernels.expert_product_tcgen05(self.raised, self.w_down, self.lowered, self.table, tiles, -1, self.rt.error_flag)
-            place = self.place
+            return self.place
+        kernels.moe_group(self.chosen, t, self.experts, top, self.place, self.source, self.table)
+        tiles = kernels.moe_max_tiles(pairs, self.experts)
+        if self.gated_experts:
+            kernels.expert_product(x, self.source, self.w_up, self.paired, self.table, tiles, -1)
+            kernels.glu(self.paired, self.raised, pairs, self.inner, self.activation, self.gate_constants)
         else:
-            kernels.moe_group(self.chosen, t, self.experts, top, self.place, self.source, self.table)
-            tiles = kernels.moe_max_tiles(pairs, self.experts)
-            kernels.expert_product(x, self.source, self.w_up, first_out, self.table, tiles, first_act)
-            if self.gated_experts:
-                kernels.glu(self.paired, self.raised, pairs, self.inner, self.activation)
-            kernels.expert_product(self.raised, None, self.w_down, self.lowered, self.table, tiles, -1)
-            place = self.place
-        kernels.moe_combine(self.lowered, place, self.weights, self.shared_out, self.shared_gate if gated else None,
-                            out, t, top)
+            kernels.expert_product(x, self.source, self.w_up, self.raised, self.table, tiles, self.activation)
+        kernels.expert_product(self.raised, None, self.w_down, self.lowered, self.table, tiles, -1)
+        return self.place
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
+        place = self._expert_rows(x, step)
+        kernels.moe_combine(self.lowered, place, self.weights, self.shared_out, self.shared_gate if self.gated else None,
+                            out, step.tokens, self.top)
+
+    def forward_terms(self, x: torch.Tensor, step: StepContext):
+        """forward() without its last sum, for a caller that forms it in a pass of its own: (rows, row of every (token,
+        choice) pair or None, float32 weights of the pairs, choices a token). None: the part has more than that to add."""
+        if self.shared is not None:
+            return None
+        return self.lowered, self._expert_rows(x, step), self.weights, self.top

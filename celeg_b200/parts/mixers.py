@@ -375,14 +375,21 @@ class PreparedAttentionMixer(PagedAttentionKernels):
 
     * biases on the projections (tensors ``q_bias``, ``k_bias``, ``v_bias``, ``out_bias``);
     * ``whole_qk_norm``: one RMS norm over the whole q projection and one over the whole k projection (tensors
-      ``q_norm``, ``k_norm`` as wide as the projections, ``eps``);
-    * a nested part ``position`` that rotates pairs (i, i + half) of the heads' leading dimensions;
+      ``q_norm``, ``k_norm`` as wide as the projections, ``eps``); or ``head_qk_norm``: one a head, with weights as wide
+      as a head that all heads share;
+    * a nested part ``position`` that rotates pairs (i, i + half), or neighbours (2i, 2i + 1), of the heads' leading
+      dimensions, with a factor on cosine and sine;
     * ``temperature`` = {coef, every}: q times 1 + coef ln(floor((position + 1) / every) + 1);
     * ``distance_far`` with the tensor ``distance_table`` [buckets, heads]: a learned number per head and distance
       bucket (:func:`distance_bucket`) added to the scaled scores;
     * ``value_mix``: "first" notes the layer's values of the step's tokens for later layers, "blend" replaces v by
       (1 - lam) v + lam v_first with lam the stored number ``value_mix`` (what is cached is the blended v);
-    * ``output_gate``: the heads' results times sigmoid(W_g h), element by element (tensor ``gate``);
+    * ``unit_values``: every value head divided by its root mean square (``eps``, no weight), and cached so;
+    * ``output_gate``: the heads' results times sigmoid(W_g h), element by element (tensor ``gate`` [heads * vdim, ...]),
+      or with "head" one number a head (tensor ``gate`` [heads, ...]);
+    * ``one_in_denominator``: the softmax's denominator holds a one beside the scores' exponentials (a sink of score 0);
+    * ``reads_cache_only``: no key and value projections; the mixer's place in the run order reads the cache of an
+      earlier one, with its own queries and everything after them;
     * values of a size ``vdim`` of their own, a softmax scale given by the configuration, a sink per head (tensor
       ``sinks``), and a mask: ``window`` = w lets a query at position i read key j when 0 <= i - j < w, ``chunk`` = c
       when floor(i / c) = floor(j / c) (chunks counted from position 0 of the sequence, so the mask does not depend
@@ -411,29 +418,49 @@ class PreparedAttentionMixer(PagedAttentionKernels):
             raise ValueError(f"attention: a window of {self.window} positions (beside a chunk: {self.chunk})")
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads are not a multiple of {self.kv_heads} kv heads")
+        self.reads_only = bool(params.get("reads_cache_only", False))
         self.sinks = rt.vector(weights["sinks"]) if "sinks" in weights else None
+        if params.get("one_in_denominator", False):
+            if self.sinks is not None:
+                raise ValueError("attention: learned sinks and a one in the denominator exclude each other")
+            self.sinks = rt.vector(torch.zeros(self.heads))
         if self.sinks is not None and self.sinks.shape != (self.heads,):
             raise ValueError(f"attention sinks have shape {tuple(self.sinks.shape)}, expected ({self.heads},)")
-        self.output_gate = bool(params.get("output_gate", False))
+        gate = params.get("output_gate", False)
+        if gate not in (None, False, True, "head"):
+            raise ValueError(f"attention: output_gate {gate!r}; known: true, head")
+        self.output_gate = bool(gate)
+        self.gate_per_head = gate == "head"
         # sizes of a stored head: what the kernels see as head size (keys, queries) and value size
         self.head_dim = self.value_dim = None
         larger = max(self.dim, self.vdim)
-        if self.dim == self.vdim or (rt.act_dtype == torch.bfloat16 and not self.output_gate
+        if self.dim == self.vdim or (rt.act_dtype == torch.bfloat16 and (self.gate_per_head or not self.output_gate)
                                      and self._fast_kernels_take(larger)):
             self.head_dim = self.value_dim = larger
         else:
             self.head_dim, self.value_dim = self.dim, self.vdim
         q_width, k_width, v_width = self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
+        if self.reads_only:
+            if {"k", "v", "k_bias", "v_bias", "k_norm"} & set(weights):
+                raise ValueError("an attention that reads another place's cache has no key and value tensors")
+            k_width = v_width = 0
         self.q_width, self.k_width, self.v_width = q_width, k_width, v_width
-        stacked = [weights["q"], weights["k"], weights["v"]]
+        stacked = [weights["q"]] if self.reads_only else [weights["q"], weights["k"], weights["v"]]
+        self.gate_width = 0
         if self.output_gate:
-            stacked.append(weights["gate"])
+            gate_rows = weights["gate"]
+            stacked.append(gate_rows)
+            self.gate_width = self.heads if self.gate_per_head else self.heads * self.vdim
+            if tuple(gate_rows.shape) != (self.gate_width, self.hidden):
+                raise ValueError(f"an output gate of shape {tuple(gate_rows.shape)}, expected ({self.gate_width}, {self.hidden})")
+            if self.gate_per_head and self.heads % 8:       # (zero rows: the projection's rows stay 16-byte aligned)
+                stacked.append(torch.zeros((-self.heads % 8, self.hidden), dtype=gate_rows.dtype))
         self.w_qkv = rt.matrix(torch.cat(stacked, dim=0))
-        self.gate_width = self.heads * self.vdim if self.output_gate else 0
         biases = [weights.get("q_bias"), weights.get("k_bias"), weights.get("v_bias")]
         if any(b is not None for b in biases):
             widths = (q_width, k_width, v_width)
-            self.bias = rt.vector(torch.cat([b.float() if b is not None else torch.zeros(w) for b, w in zip(biases, widths)]))
+            self.bias = rt.vector(torch.cat([b.float() if b is not None else torch.zeros(w)
+                                             for b, w in zip(biases, widths)]))
         else:
             self.bias = None
         # what the plain store (biases only) cannot do goes through the general preparation
@@ -445,13 +472,24 @@ class PreparedAttentionMixer(PagedAttentionKernels):
             if self.q_norm.shape != (q_width,) or self.k_norm.shape != (k_width,):
                 raise ValueError(f"whole-projection norm weights of shapes {tuple(self.q_norm.shape)} / "
                                  f"{tuple(self.k_norm.shape)}, expected ({q_width},) / ({k_width},)")
+        self.head_qk_norm = bool(params.get("head_qk_norm", False))
+        if self.head_qk_norm:
+            if self.whole_qk_norm:
+                raise ValueError("attention: whole_qk_norm and head_qk_norm exclude each other")
+            self.q_norm = rt.vector(weights["q_norm"])
+            self.k_norm = None if self.reads_only else rt.vector(weights["k_norm"])
+            for vector in (self.q_norm, self.k_norm):
+                if vector is not None and vector.shape != (self.dim,):
+                    raise ValueError(f"a head norm's weight has shape {tuple(vector.shape)}, expected ({self.dim},)")
+        self.unit_values = bool(params.get("unit_values", False)) and not self.reads_only
         position = parts.get("position")
         fused = position.fused() if position is not None else None
-        self.frequencies, self.rotary_dim = None, 0
+        self.frequencies, self.rotary_dim, self.interleaved, self.magnitude = None, 0, False, 1.0
         if fused is not None and fused.get("rotary_dim"):
-            if fused.get("interleaved") or fused["rotary_dim"] > self.dim:
-                raise ValueError("attention: the position part must rotate pairs (i, i + half) of at most dim dimensions")
+            if fused["rotary_dim"] > self.dim:
+                raise ValueError("attention: the position part must rotate at most dim dimensions")
             self.frequencies, self.rotary_dim = fused["inv_freq"], int(fused["rotary_dim"])
+            self.interleaved, self.magnitude = bool(fused.get("interleaved")), float(fused.get("magnitude", 1.0))
         elif position is not None and fused is None:
             raise ValueError("attention: the position part must offer fused() tables")
         temperature = params.get("temperature")
@@ -467,11 +505,14 @@ class PreparedAttentionMixer(PagedAttentionKernels):
         mix = params.get("value_mix")
         if mix not in (None, "first", "blend"):
             raise ValueError(f"attention: value_mix {mix!r}; known: first, blend")
+        if mix is not None and self.reads_only:
+            raise ValueError("attention: values cannot be blended by a mixer that has none of its own")
         self.blend = {None: 0, "first": 1, "blend": 2}[mix]
         self.lam = float(weights["value_mix"].to(torch.float32).reshape(-1)[0]) if self.blend == 2 else 0.0
         # the first marked layer's values of the step's tokens: float32 rows that every marked layer of a model shares
         self.first_values = rt.scratch("attention.first_values", v_width, torch.float32) if self.blend else None
-        self.prepares = bool(self.whole_qk_norm or self.frequencies is not None or self.temperature or self.blend)
+        self.prepares = bool(self.whole_qk_norm or self.head_qk_norm or self.frequencies is not None or self.temperature
+                             or self.blend or self.unit_values or self.reads_only)
         w_out = weights["out"]
         if self.value_dim != self.vdim:          # zero columns where the attention's result has its zero tail
             padded = torch.zeros((w_out.shape[0], self.heads, self.value_dim), dtype=w_out.dtype)
@@ -482,7 +523,7 @@ class PreparedAttentionMixer(PagedAttentionKernels):
         self.ends_with_product = self.out_bias is None       # forward() then writes `out` last, with rt.linear
         self.binding: Optional[PagedBinding] = None
         self._resident_blocks: Optional[int] = None
-        self.projected = rt.scratch("prepared_attention.proj", q_width + k_width + v_width + self.gate_width, torch.float32)
+        self.projected = rt.scratch("prepared_attention.proj", int(self.w_qkv.shape[0]), torch.float32)
         self.qkv_width = self.heads * self.head_dim
         self.qkv = rt.scratch("prepared_attention.q", self.qkv_width)
         self.attended = rt.scratch("prepared_attention.out", self.heads * self.value_dim)
@@ -497,8 +538,9 @@ class PreparedAttentionMixer(PagedAttentionKernels):
                          value_head_dim=None if self.value_dim == self.head_dim else self.value_dim)
 
     def bind_cache(self, binding: PagedBinding) -> None:
-        if not binding.owner:
-            raise ValueError("this attention writes its keys and values: it cannot read another position's cache")
+        if binding.owner == self.reads_only:
+            raise ValueError("an attention without key and value projections cannot own a cache" if binding.owner else
+                             "this attention writes its keys and values: it cannot read another position's cache")
         self.binding = binding
 
     def _attend(self, x: torch.Tensor, step: StepContext) -> None:
@@ -506,10 +548,13 @@ class PreparedAttentionMixer(PagedAttentionKernels):
         rt.linear(x, self.w_qkv, self.projected, t)
         table = step.block_tables[b.group]
         if self.prepares:
-            kernels.qkv_prepare(self.projected, self.bias, self.qkv, step.positions, step.token_span, table, b.k, b.v, t,
-                                self.heads, self.kv_heads, self.dim, self.vdim, self.head_dim, self.value_dim,
+            k_pages, v_pages, kv_heads = (None, None, 0) if self.reads_only else (b.k, b.v, self.kv_heads)
+            kernels.qkv_prepare(self.projected, self.bias, self.qkv, step.positions, step.token_span, table, k_pages, v_pages,
+                                t, self.heads, kv_heads, self.dim, self.vdim, self.head_dim, self.value_dim,
                                 b.page_tokens, step.error_flag, q_norm=self.q_norm, k_norm=self.k_norm,
-                                norm_eps=self.eps, frequencies=self.frequencies, rotary_dim=self.rotary_dim,
+                                norm_eps=self.eps, norm_per_head=self.head_qk_norm,
+                                unit_values_eps=self.eps if self.unit_values else None, frequencies=self.frequencies,
+                                rotary_dim=self.rotary_dim, interleaved=self.interleaved, magnitude=self.magnitude,
                                 temperature=self.temperature, blend=self.blend, lam=self.lam,
                                 first_values=self.first_values)
         else:
@@ -518,8 +563,9 @@ class PreparedAttentionMixer(PagedAttentionKernels):
                                   b.page_tokens, step.error_flag)
         self.attend(step, table)
         if self.output_gate:
-            kernels.sigmoid_gate(self.attended, self.projected[:, self.q_width + self.k_width + self.v_width:], t,
-                                 self.gate_width)
+            at = self.q_width + self.k_width + self.v_width
+            kernels.sigmoid_gate(self.attended, self.projected[:, at:at + self.gate_width], t, self.heads * self.value_dim,
+                                 self.value_dim if self.gate_per_head else 1)
 
     def forward_without_bias(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> Optional[torch.Tensor]:
         """forward() into a float32 ``out`` without the output projection's bias, which is returned (or None) for a

@@ -13,6 +13,8 @@ float32 results.
                   (Sun et al., "Retentive Network: A Successor to Transformer for Large Language Models", 2023)
     lightning_attention   the same recurrence with SiLU on q, k and v and no factor on the keys; the heads' read-outs
                   are normalised together, as one vector, and gated by a sigmoid
+    general_delta   S' = diag(w) S - (a u)(u^T S) + k v^T with a decay w and a removal rate a per key channel, u the unit
+                  key, read-out S'^T r (kernels: csrc/general_delta.cu)
 """
 from __future__ import annotations
 
@@ -411,3 +413,83 @@ class GatedLinearRecurrenceMixer:
                              self.result, self.state, b.slot_stride, step.span_begin, step.span_slot, t, step.spans,
                              width)
         rt.linear(self.result, self.w_out, out, t)
+
+
+@register_part("mixer", "general_delta")
+class GeneralDeltaMixer:
+    """r = W_r x, k = W_k x, v = W_v x (heads x dim each). Per key channel a decay w = exp(-e^(-1/2) sigmoid(W_2 tanh(W_1 x)
+    + w0)) and a removal rate a = sigmoid(W_a x + b_a); with the unit key u = k / sqrt(sum(k^2) + 1e-6) of each head
+    S <- diag(w) S - (a u)(u^T S) + k v^T, both terms of the old state, and the read-out S^T r of the new one. Each head's
+    read-out is divided by its root mean square, scaled by ``norm`` (all heads' width), gated by sigmoid(W_g x) and
+    projected by W_o. Per-request state: S per head, float32, zero for a new request.
+
+    One fused [r | k | v | gate | removal | W_1] projection leaves float32 sums. Decoding: one launch between the two
+    projections. Portions: tanh and the product with W_2, then the recurrence in chunks of eight tokens, then the heads'
+    norm and gate. The rank of W_2 W_1 is padded with zero rows and columns to a multiple of eight (tanh(0) = 0)."""
+
+    UNIT_EPS = 1e-6
+
+    def __init__(self, params: Mapping, weights: Mapping[str, torch.Tensor], parts: Mapping, rt: Runtime):
+        self.rt = rt
+        self.hidden = int(params["hidden_size"])
+        self.heads = int(params["heads"])
+        self.dim = int(params["dim"])
+        self.eps = float(params["eps"])
+        if self.dim > kernels.SCAN_MAX_DIM:
+            raise ValueError(f"general_delta: a head size of {self.dim} exceeds {kernels.SCAN_MAX_DIM}")
+        inner = self.inner = self.heads * self.dim
+        down, up = weights["decay_down"], weights["decay_up"]
+        rank = int(down.shape[0])
+        self.rank = -(-rank // 8) * 8
+        if self.rank != rank:
+            down = torch.cat([down, torch.zeros((self.rank - rank, down.shape[1]), dtype=down.dtype)], dim=0)
+            up = torch.cat([up, torch.zeros((up.shape[0], self.rank - rank), dtype=up.dtype)], dim=1)
+        self.w_in = rt.matrix(torch.cat([weights["r"], weights["k"], weights["v"], weights["gate"], weights["removal"], down],
+                                        dim=0))
+        self.w_decay = rt.matrix(up)
+        self.w_out = rt.matrix(weights["out"])
+        self.removal_bias = rt.vector(weights["removal_bias"])
+        self.decay_bias = rt.vector(weights["decay_bias"])
+        self.norm = rt.vector(weights["norm"])
+        for name, vector in (("removal_bias", self.removal_bias), ("decay_bias", self.decay_bias), ("norm", self.norm)):
+            if vector.shape != (inner,):
+                raise ValueError(f"general_delta: {name} has shape {tuple(vector.shape)}, expected ({inner},)")
+        self.binding: Optional[StateBinding] = None
+        self.projected = rt.scratch("recurrent.proj", int(self.w_in.shape[0]), torch.float32)
+        self.low = rt.scratch("general_delta.low", self.rank)
+        self.z = rt.scratch("general_delta.z", inner, torch.float32)
+        pad = self.heads * (-(-self.dim // 4) * 4)
+        self.vectors = rt.flat_scratch("general_delta.vectors", rt.max_tokens * 4 * pad, torch.float32)
+        self.chunk_decay = rt.flat_scratch("general_delta.decay", rt.max_tokens * pad, torch.float32)
+        self.sums = rt.flat_scratch("general_delta.sums", rt.max_tokens * self.heads * 2 * kernels.DELTA_CHUNK, torch.float32)
+        self.read = rt.scratch("recurrent.read", inner, torch.float32)
+        self.gated = rt.scratch("recurrent.gated", inner)
+
+    def cache_need(self):
+        return StateNeed(elements=self.heads * self.dim * self.dim)
+
+    def bind_cache(self, binding: StateBinding) -> None:
+        self.binding = binding
+
+    ends_with_product = True      # forward() writes `out` last, with rt.linear
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
+        rt, t, b, inner = self.rt, step.tokens, self.binding, self.inner
+        rt.linear(x, self.w_in, self.projected, t)
+        rows = self.projected
+        if step.max_span == 1 and step.spans == t:
+            # every request brings one token
+            kernels.general_delta_decode(rows, (0, inner, 2 * inner, 3 * inner, 4 * inner, 5 * inner), self.w_decay,
+                                         self.decay_bias, self.removal_bias, self.norm, self.eps, self.UNIT_EPS, b.state,
+                                         b.slot_stride, step.span_slot, t, self.heads, self.dim, self.gated)
+            rt.linear(self.gated, self.w_out, out, t)
+            return
+        kernels.activation_cast(rows[:, 5 * inner:], self.low, t, kernels.ACT_TANH)
+        rt.linear(self.low, self.w_decay, self.z, t)
+        kernels.general_delta_scan(rows, (0, inner, 2 * inner, 4 * inner), self.z, self.decay_bias, self.removal_bias,
+                                   self.UNIT_EPS, step.token_span, step.span_begin, step.span_slot, self.vectors,
+                                   self.chunk_decay, self.sums, self.read, b.state, b.slot_stride, t, step.spans, self.heads,
+                                   self.dim)
+        kernels.gated_head_norm(self.read, rows[:, 3 * inner:4 * inner], self.norm, True, self.gated, t, self.heads, self.dim,
+                                self.eps, kernels.GATE_SIGMOID)
+        rt.linear(self.gated, self.w_out, out, t)

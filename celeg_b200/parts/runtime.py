@@ -45,6 +45,11 @@ class ResidualStream:
         # stream part that runs after a block may write that norm's output itself and say so in ``ready``
         self.upcoming = None
         self.ready = None
+        # blocks whose sublayers read the stream itself: its rows in the activation type (on the float32 path the
+        # stream's own), whether they are those of the stream as it is now, and whether the first block wants them
+        self.rows = rt.scratch("stream.rows", hidden) if rt.act_dtype != torch.float32 else self.residual
+        self.rows_current = False
+        self.wants_rows = False
         self.pieces = (hidden + 15) // 16
         if rt.act_dtype == torch.bfloat16:
             self.xw = rt.scratch("stream.split_norm", hidden, torch.bfloat16)
@@ -57,7 +62,38 @@ class ResidualStream:
         self.after_layer = None
         self.upcoming = None
         self.ready = None
+        self.rows_current = False
         self.rt.sink = None
+
+    def as_rows(self, rows: int) -> torch.Tensor:
+        """The stream's first ``rows`` rows in the activation type, with everything owed to it added: what a sublayer
+        without a norm before it reads."""
+        if self.prepared is not None:
+            raise RuntimeError("a norm was prepared for another reader than one that wants the stream itself")
+        if self.pending is not None or self.pending_b is not None:
+            self.settle(rows)
+        if self.rows is not self.residual and not self.rows_current:
+            kernels.output_norm(self.residual, rows, None, None, 0.0, self.rows)
+        self.rows_current = True
+        return self.rows
+
+    def add_normed(self, norm, rows: int, output: torch.Tensor, *, place: Optional[torch.Tensor] = None,
+                   weights: Optional[torch.Tensor] = None, top: int = 1, bias: Optional[torch.Tensor] = None,
+                   upcoming=None) -> None:
+        """stream += norm(y) for good, y = output (+ bias) or the weighted sum of ``top`` of its rows a token (see
+        kernels.output_norm), in the pass that also leaves what is read next: the stream's rows in the activation type,
+        or the first half of the norm ``upcoming`` where its reader takes a split norm."""
+        weight, eps = norm.as_prologue()
+        halves = self.split(upcoming, 1) if upcoming is not None and self.rt.small_batch(rows) else None
+        if halves is not None:
+            kernels.output_norm(self.residual, rows, output, weight, eps, None, place=place, weights=weights, top=top,
+                                bias=bias, prepare=halves[1], next_weight=halves[0])
+            self.prepared = (upcoming, halves[1])
+            self.rows_current = False
+            return
+        kernels.output_norm(self.residual, rows, output, weight, eps, None if self.rows is self.residual else self.rows,
+                            place=place, weights=weights, top=top, bias=bias)
+        self.rows_current = True
 
     def split(self, norm, pieces: int):
         """(weight, SplitNorm) for a norm that can be split, else None."""
@@ -111,8 +147,13 @@ class ResidualStream:
     def settle(self, rows: int) -> None:
         """Add what is owed to the stream now (for a reader that wants the stream itself)."""
         if self.pending is not None or self.pending_b is not None:
+            self.rows_current = False
             kernels.add_to_residual(self.residual, self.pending, self.pending_b, rows)
             self.pending = self.pending_b = None
+
+    def changed(self) -> None:
+        """A part has rewritten the stream itself."""
+        self.rows_current = False
 
     def expect(self, buffer: torch.Tensor, upcoming, rows: int) -> None:
         """A part is about to write its output to ``buffer``; ``upcoming`` is the norm that reads the
@@ -127,6 +168,7 @@ class ResidualStream:
 
     def add_later(self, delta: torch.Tensor) -> None:
         assert self.pending is None
+        self.rows_current = False
         sink, self.rt.sink = self.rt.sink, None
         if sink is not None and sink.used:
             self.prepared = (sink.norm, sink.split)          # the product has added to the stream already

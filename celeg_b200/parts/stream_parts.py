@@ -40,6 +40,7 @@ class EmbeddingReentry:
         kernels.join_stream_embedding(stream.residual, stream.pending, stream.pending_b, self.table,
                                       step.token_ids[:t], self.joined, t, self.multiplier)
         stream.pending = stream.pending_b = None
+        stream.changed()
         self.rt.linear(self.joined, self.weight, stream.residual, t)
 
 
@@ -81,3 +82,4 @@ class DepthAverage:
             kernels.depth_average(stream.residual, stream.pending, stream.pending_b, self.history, self.weights,
                                   self.index, t)
         stream.pending = stream.pending_b = None
+        stream.changed()
