@@ -199,7 +199,7 @@ class KernelTimer:
              "expert_product", "expert_product_tcgen05", "expert_rows", "moe_combine", "retention_segmented",
              "retention_decode_raw", "activation_columns", "bias_store_kv", "scaled_sum", "glu", "lru_prepare",
              "block_diagonal_product", "lru_scan", "lru_decode", "add_layernorm", "qkv_prepare", "rmsnorm_strided",
-             "sigmoid_gate")
+             "sigmoid_gate", "output_norm", "activation_cast", "general_delta_scan", "general_delta_decode")
 
     def __init__(self):
         self.pairs = []

@@ -38,7 +38,8 @@ constexpr int kDeltaMaxDim = 256;
 constexpr float kDecaySpan = 0.60653065971263342f;             // e^(-1/2)
 
 __device__ __forceinline__ float sigmoid_of(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float channel_decay(float z) { return expf(-kDecaySpan * sigmoid_of(z)); }
+// 1 + expm1: a decay close to one is then its nearest float, without a bias that thousands of steps would add up
+__device__ __forceinline__ float channel_decay(float z) { return 1.0f + expm1f(-kDecaySpan * sigmoid_of(z)); }
 
 struct DeltaVectorsArgs {
     const float* proj; int stride; int r_off, k_off, a_off;    // columns of a token's row: head h at h * dim
