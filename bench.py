@@ -8,7 +8,7 @@ batch 1 and 64. Prints ONE JSON line.
                   [--prefill-tokens T] [--chunk C] [--kernel-times] [--no-cuda-graph]      one phase, a short record
   python bench.py --workload lfm2-700m|lfm2-350m [--requests N] [--new-tokens N] [--max-batched-tokens N]
                   [--prefill-chunk N] [--kernel-times]       a scheduler workload through Engine.submit/step/poll
-  python bench.py --design ramosun|kedesun|naselorn|liverax [--design-size w1024|w2048] [--kernel-times]
+  python bench.py --design ramosun|kedesun|naselorn|liverax|kodupel [--design-size w1024|w2048] [--kernel-times]
                   the Ramosun design beside the closest LFM2 model at equal size: prefill of 2,048 tokens, decode at batch 8
 
 A "step" is one decode step of the whole batch. ``value`` is timed on the device (CUDA events
@@ -543,6 +543,25 @@ def liverax_config(width: int, vocab: int) -> dict:
             "layers": run + run, "distance_buckets": [0, 0, 0, 32] * 2, "max_context": 8192}
 
 
+def kodupel_config(width: int, vocab: int) -> dict:
+    """Eight layers, each with experts: the generalised delta rule, rotary attention, attention over that layer's keys and
+    values, the delta rule, twice. Heads of 64 (width / 64 of them) in both mixers, a quarter as many key heads; decay
+    projections of rank width / 32; 24 gated experts of half the width of which a token uses 4 (as many parameters as
+    Naselorn's four mixtures of 32 with their shared experts and four dense feed-forwards)."""
+    heads = width // 64
+    experts = {"kind": "moe", "router": {"experts": 24, "top": 4}, "expert": {"ff": width // 2, "limit": 7.0}}
+    delta = {"type": "general_delta", "mlp": experts, "mixer": {"heads": heads, "dim": 64, "decay_rank": width // 32}}
+
+    def attention(kv_from=None):
+        mixer = {"heads": heads, "kv_heads": heads // 4, "dim": 64, "vdim": 64, "scale": 0.125, "rot": {
+            "base": 500000.0, "dims": 32, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+        return {"type": "attention", "mlp": experts, "mixer": mixer if kv_from is None else dict(mixer, kv_from=kv_from)}
+
+    layers = [delta, attention(), attention(1), delta, delta, attention(), attention(5), delta]
+    return {"architecture": "Kodupel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 4.0},
+            "layers": layers, "max_context": 8192}
+
+
 def lfm2_attention_only(width: int, vocab: int) -> dict:
     """The LFM2 relative with attention in all eight blocks: the existing model closest to a design whose mixers are all
     softmax attention (pre-norm blocks, grouped queries, rotation of halves, a gated feed-forward)."""
@@ -582,6 +601,9 @@ def run_design(args) -> dict:
         elif args.design == "liverax":   # beside LFM2 with attention in every block, and Kedesun for the latent mixer
             models = (("liverax", liverax_config(width, vocab)), ("lfm2_attention", lfm2_attention_only(width, vocab)),
                       ("kedesun", kedesun_config(width, vocab)))
+        elif args.design == "kodupel":   # beside Naselorn (gated experts) and Ramosun (a delta rule, per-head state)
+            models = (("kodupel", kodupel_config(width, vocab)), ("naselorn", naselorn_config(width, vocab)),
+                      ("ramosun", ramosun_config(width, vocab)))
         else:
             models = (("ramosun", ramosun_config(width, vocab)), ("lfm2", lfm2_relative(width, vocab)))
         for name, raw in models:
@@ -863,7 +885,7 @@ def main() -> int:
     parser.add_argument("--new-tokens", type=int, default=0, help="--workload: tokens to generate per request")
     parser.add_argument("--max-batched-tokens", type=int, default=0, help="--workload: token budget of a step")
     parser.add_argument("--prefill-chunk", type=int, default=0, help="--workload: longest prompt portion")
-    parser.add_argument("--design", default=None, choices=["ramosun", "kedesun", "naselorn", "liverax"],
+    parser.add_argument("--design", default=None, choices=["ramosun", "kedesun", "naselorn", "liverax", "kodupel"],
                         help="prefill and decode of that design beside the closest LFM2 model at equal size")
     parser.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="--design: one size only")
     parser.add_argument("--no-warmup-run", action="store_true",

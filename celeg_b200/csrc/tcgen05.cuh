@@ -72,6 +72,13 @@ __device__ __forceinline__ void tma_load_2d(unsigned smem_dst, const CUtensorMap
         : "memory");
 }
 
+// An untiled copy of `bytes` (a multiple of 16) from and to 16-byte aligned addresses, counted by the mbarrier.
+__device__ __forceinline__ void bulk_load(unsigned smem_dst, const void* src, unsigned bytes, unsigned bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n" ::"r"(smem_dst),
+                 "l"(src), "r"(bytes), "r"(bar)
+                 : "memory");
+}
+
 __device__ __forceinline__ void tmem_alloc(unsigned smem_result, unsigned columns) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_result), "r"(columns)
                  : "memory");

@@ -61,9 +61,10 @@ _SIGNATURES = {
                           c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "celeg_embedding_copy": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "celeg_activation_cast": [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_general_delta_scratch": [c_int, c_int],
     "celeg_general_delta_scan": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float,
-                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong,
-                                 c_int, c_int, c_int, c_int, c_void_p],
+                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int,
+                                 c_int, c_void_p, c_void_p],
     "celeg_general_delta_decode": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
                                    c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int,
                                    c_void_p, c_int, c_void_p],
@@ -947,9 +948,6 @@ def retention_decode_raw(proj: torch.Tensor, offsets: Tuple[int, int, int], deca
 
 
 # ------------------------------------------------------------------------------- generalised delta rule
-DELTA_CHUNK = 8             # tokens whose sums over the state are formed together (csrc/general_delta.cu)
-
-
 def activation_cast(x: torch.Tensor, out: torch.Tensor, tokens: int, kind: int) -> None:
     """out[:tokens] = act(x[:tokens]) of float32 columns that lie in wider rows, rounded once to the type of ``out``."""
     assert x.dtype == torch.float32 and x.stride(-1) == 1 and out.is_contiguous() and x.shape[-1] == out.shape[-1]
@@ -957,24 +955,26 @@ def activation_cast(x: torch.Tensor, out: torch.Tensor, tokens: int, kind: int) 
                                            dtype_code(out.dtype), _stream()))
 
 
+def general_delta_scratch(heads: int, dim: int) -> int:
+    """Floats of scratch a token that :func:`general_delta_scan` needs."""
+    return int(library().celeg_general_delta_scratch(heads, dim))
+
+
 def general_delta_scan(proj: torch.Tensor, offsets: Tuple[int, int, int, int], z: torch.Tensor, w0: torch.Tensor,
                        a_bias: torch.Tensor, unit_eps: float, token_span: torch.Tensor, span_begin: torch.Tensor,
-                       span_slot: torch.Tensor, vectors: torch.Tensor, decay: torch.Tensor, sums: torch.Tensor,
-                       out: torch.Tensor, state: torch.Tensor, slot_stride: int, tokens: int, spans: int, heads: int,
-                       dim: int) -> None:
-    """S <- diag(w) S - b (u^T S) + k v^T, o = S^T r along the step's spans (csrc/general_delta.cu). ``offsets``: columns of
-    (r, k, v, removal rate) in a row of ``proj``; ``z`` [>= tokens, heads * dim] the decay before its bias ``w0``. Scratch,
-    all float32: ``vectors`` tokens * heads * 4 * dim', ``decay`` tokens * heads * dim', ``sums`` heads * tokens * 16
-    elements, dim' = dim rounded up to a multiple of 4."""
-    pad = -(-dim // 4) * 4
-    for tensor in (proj, z, w0, a_bias, vectors, decay, sums, out, state):
+                       span_slot: torch.Tensor, records: torch.Tensor, out: torch.Tensor, state: torch.Tensor,
+                       slot_stride: int, tokens: int, spans: int, heads: int, dim: int, error_flag: torch.Tensor) -> None:
+    """S <- diag(w) S - b (u^T S) + k v^T, o = S^T r along the step's spans (csrc/general_delta_scan.cu). ``offsets``:
+    columns of (r, k, v, removal rate) in a row of ``proj``; ``z`` [>= tokens, heads * dim] the decay before its bias
+    ``w0``; ``records``: float32 scratch of tokens * :func:`general_delta_scratch` elements."""
+    for tensor in (proj, z, w0, a_bias, records, out, state):
         assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
-    assert vectors.numel() >= tokens * heads * 4 * pad and decay.numel() >= tokens * heads * pad
-    assert sums.numel() >= heads * tokens * 2 * DELTA_CHUNK and out.is_contiguous() and out.shape[1] == heads * dim
+    assert records.numel() >= tokens * general_delta_scratch(heads, dim)
+    assert out.is_contiguous() and out.shape[1] == heads * dim
     _check(library().celeg_general_delta_scan(
         _ptr(proj), proj.stride(0), *offsets, _ptr(z), z.stride(0), _ptr(w0), _ptr(a_bias), unit_eps, _ptr(token_span),
-        _ptr(span_begin), _ptr(span_slot), _ptr(vectors), _ptr(decay), _ptr(sums), _ptr(out), _ptr(state), slot_stride,
-        tokens, spans, heads, dim, _stream()))
+        _ptr(span_begin), _ptr(span_slot), _ptr(records), _ptr(out), _ptr(state), slot_stride, tokens, spans, heads, dim,
+        _ptr(error_flag), _stream()))
     global LAUNCHES
     LAUNCHES += 1          # the vectors, then the scan
 

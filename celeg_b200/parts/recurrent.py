@@ -14,7 +14,7 @@ float32 results.
     lightning_attention   the same recurrence with SiLU on q, k and v and no factor on the keys; the heads' read-outs
                   are normalised together, as one vector, and gated by a sigmoid
     general_delta   S' = diag(w) S - (a u)(u^T S) + k v^T with a decay w and a removal rate a per key channel, u the unit
-                  key, read-out S'^T r (kernels: csrc/general_delta.cu)
+                  key, read-out S'^T r (kernels: csrc/general_delta_scan.cu, csrc/general_delta.cu)
 """
 from __future__ import annotations
 
@@ -458,10 +458,8 @@ class GeneralDeltaMixer:
         self.projected = rt.scratch("recurrent.proj", int(self.w_in.shape[0]), torch.float32)
         self.low = rt.scratch("general_delta.low", self.rank)
         self.z = rt.scratch("general_delta.z", inner, torch.float32)
-        pad = self.heads * (-(-self.dim // 4) * 4)
-        self.vectors = rt.flat_scratch("general_delta.vectors", rt.max_tokens * 4 * pad, torch.float32)
-        self.chunk_decay = rt.flat_scratch("general_delta.decay", rt.max_tokens * pad, torch.float32)
-        self.sums = rt.flat_scratch("general_delta.sums", rt.max_tokens * self.heads * 2 * kernels.DELTA_CHUNK, torch.float32)
+        self.records = rt.flat_scratch("general_delta.records",
+                                       rt.max_tokens * kernels.general_delta_scratch(self.heads, self.dim), torch.float32)
         self.read = rt.scratch("recurrent.read", inner, torch.float32)
         self.gated = rt.scratch("recurrent.gated", inner)
 
@@ -487,9 +485,8 @@ class GeneralDeltaMixer:
         kernels.activation_cast(rows[:, 5 * inner:], self.low, t, kernels.ACT_TANH)
         rt.linear(self.low, self.w_decay, self.z, t)
         kernels.general_delta_scan(rows, (0, inner, 2 * inner, 4 * inner), self.z, self.decay_bias, self.removal_bias,
-                                   self.UNIT_EPS, step.token_span, step.span_begin, step.span_slot, self.vectors,
-                                   self.chunk_decay, self.sums, self.read, b.state, b.slot_stride, t, step.spans, self.heads,
-                                   self.dim)
+                                   self.UNIT_EPS, step.token_span, step.span_begin, step.span_slot, self.records,
+                                   self.read, b.state, b.slot_stride, t, step.spans, self.heads, self.dim, step.error_flag)
         kernels.gated_head_norm(self.read, rows[:, 3 * inner:4 * inner], self.norm, True, self.gated, t, self.heads, self.dim,
                                 self.eps, kernels.GATE_SIGMOID)
         rt.linear(self.gated, self.w_out, out, t)

@@ -139,15 +139,16 @@ def test_delta_scan_over_spans_of_all_lengths(heads, dim, lengths, slow):
     low = np.tanh(case.proj[:, case.offsets[5]:].astype(np.float64))
     want, want_state = case.expected(low)
     z = gpu(low @ case.up.T)
-    pad = heads * (-(-dim // 4) * 4)
+    flag = torch.zeros(1, dtype=torch.int32, device=DEVICE)
     state = gpu(case.state)
     read = torch.full((tokens, inner), 7.0, dtype=torch.float32, device=DEVICE)
     spans = np.repeat(np.arange(len(lengths)), lengths)
     filled = lambda n: torch.full((n,), float("nan"), dtype=torch.float32, device=DEVICE)
     k.general_delta_scan(gpu(case.proj), (case.offsets[0], case.offsets[1], case.offsets[2], case.offsets[4]), z, gpu(case.w0),
                          gpu(case.a_bias), 1e-6, gpu(spans, torch.int32), gpu(case.begin, torch.int32),
-                         gpu(case.slots, torch.int32), filled(tokens * 4 * pad), filled(tokens * pad), filled(tokens * heads * 16),
-                         read, state, case.stride, tokens, len(lengths), heads, dim)
+                         gpu(case.slots, torch.int32), filled(tokens * k.general_delta_scratch(heads, dim)), read, state,
+                         case.stride, tokens, len(lengths), heads, dim, flag)
+    assert int(flag.item()) == 0
     close(read, want, 3e-5, "read-outs")
     close(state, want_state, 3e-5, "states")
     untouched = np.setdiff1d(np.arange(case.state.shape[0]), case.slots)
