@@ -183,6 +183,113 @@ __global__ void qkv_prepare_kernel(const QkvPrepareArgs p) {
     }
 }
 
+// The same for rows whose heads need nothing from one another (norms per head or none, pairs of neighbours or no rotation,
+// no query factor, no blending, heads stored as wide as they are): a warp a head straight from and to memory, a pair of
+// neighbours a lane, angles once a warp, no shared memory and no barrier. E: pairs a lane (heads of up to 64 E entries).
+template <typename A> __device__ __forceinline__ void store_pair(A* p, float x, float y);
+template <> __device__ __forceinline__ void store_pair<float>(float* p, float x, float y) {
+    *reinterpret_cast<float2*>(p) = make_float2(x, y);
+}
+template <> __device__ __forceinline__ void store_pair<__nv_bfloat16>(__nv_bfloat16* p, float x, float y) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y);
+}
+
+template <typename A, int E>
+__global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepareArgs p) {
+    constexpr int kAhead = 4;                              // heads whose loads are under way together
+    chain_release();
+    chain_wait();
+    const int t = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int pos = p.positions[t];
+    const int page = p.kv_heads > 0 ? p.block_table[(size_t)p.token_span[t] * p.table_stride + pos / p.page_tokens] : 0;
+    const int in_page = pos % p.page_tokens;
+    const int half = p.frequencies ? p.rotary_dim >> 1 : 0;
+    const int q_width = p.q_heads * p.head_dim, qk_width = q_width + p.kv_heads * p.head_dim;
+    const float* row = p.proj + (size_t)t * p.proj_stride;
+    if (page < 0 && threadIdx.x == 0) atomicExch(p.error_flag, 2);
+    float c[E], s[E];
+#pragma unroll
+    for (int x = 0; x < E; ++x) {
+        c[x] = 1.0f;
+        s[x] = 0.0f;
+        const int pair = lane + 32 * x;
+        if (pair < half) {
+            sincosf((float)pos * p.frequencies[pair], &s[x], &c[x]);
+            c[x] *= p.magnitude;
+            s[x] *= p.magnitude;
+        }
+    }
+    const int units = p.q_heads + 2 * p.kv_heads;
+    for (int base = warp; base < units; base += kAhead * warps) {
+        float2 v[kAhead][E];
+#pragma unroll
+        for (int a = 0; a < kAhead; ++a) {
+            const int unit = base + a * warps;
+            const bool value = unit >= p.q_heads + p.kv_heads;
+            const int at = value ? qk_width + (unit - p.q_heads - p.kv_heads) * p.value_dim : unit * p.head_dim;
+#pragma unroll
+            for (int x = 0; x < E; ++x) {
+                const int e = 2 * (lane + 32 * x);
+                v[a][x] = make_float2(0.0f, 0.0f);
+                if (unit < units && e < (value ? p.value_dim : p.head_dim)) {
+                    v[a][x] = *reinterpret_cast<const float2*>(row + at + e);
+                    if (p.bias) {
+                        const float2 b = __ldg(reinterpret_cast<const float2*>(p.bias + at + e));
+                        v[a][x].x += b.x;
+                        v[a][x].y += b.y;
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int a = 0; a < kAhead; ++a) {
+            const int unit = base + a * warps;
+            if (unit >= units) continue;                   // (the same for the whole warp)
+            const bool is_q = unit < p.q_heads, value = unit >= p.q_heads + p.kv_heads;
+            const int size = value ? p.value_dim : p.head_dim;
+            const float* weight = value ? nullptr : is_q ? p.q_norm_w : p.k_norm_w;
+            float factor = 1.0f;
+            if (weight || (value && p.unit_values)) {
+                float squares = 0.0f;
+#pragma unroll
+                for (int x = 0; x < E; ++x) squares += v[a][x].x * v[a][x].x + v[a][x].y * v[a][x].y;
+                factor = 1.0f / sqrtf(warp_sum(squares) / (float)size + (value ? p.value_eps : p.norm_eps));
+            }
+            A* dst;
+            if (is_q) {
+                dst = static_cast<A*>(p.q_out) + (size_t)t * p.q_stride + (size_t)unit * p.head_dim;
+            } else {
+                if (page < 0) continue;
+                const int head = unit - p.q_heads - (value ? p.kv_heads : 0);
+                dst = value ? static_cast<A*>(p.v_cache) + (long long)page * p.value_page_stride
+                            : static_cast<A*>(p.k_cache) + (long long)page * p.page_stride;
+                dst += ((long long)head * p.page_tokens + in_page) * size;
+            }
+#pragma unroll
+            for (int x = 0; x < E; ++x) {
+                const int e = 2 * (lane + 32 * x);
+                if (e >= size) continue;
+                float u = v[a][x].x * factor, w = v[a][x].y * factor;
+                if (weight) {
+                    const float2 scale = __ldg(reinterpret_cast<const float2*>(weight + e));
+                    u *= scale.x;
+                    w *= scale.y;
+                }
+                if (value || lane + 32 * x >= half) store_pair<A>(dst + e, u, w);
+                else store_pair<A>(dst + e, u * c[x] - w * s[x], w * c[x] + u * s[x]);
+            }
+        }
+    }
+}
+
+template <typename A>
+static void launch_prepare_heads(const QkvPrepareArgs& args, int tokens, cudaStream_t stream) {
+    const int size = args.head_dim > args.value_dim ? args.head_dim : args.value_dim;
+    if (size <= 64) launch_chained(qkv_prepare_heads_kernel<A, 1>, tokens, 128, 0, stream, args);
+    else launch_chained(qkv_prepare_heads_kernel<A, 2>, tokens, 128, 0, stream, args);
+}
+
 }  // namespace celeg_b200
 
 using namespace celeg_b200;
@@ -222,6 +329,17 @@ CELEG_API int celeg_qkv_prepare(const float* proj, int proj_stride, const float*
                                  temp_every, blend, lam, first_values, first_stride, q_out, q_stride, positions, token_span, block_table, table_stride, k_cache, v_cache, page_stride,
                                  value_page_stride, q_heads, kv_heads, head_dim, value_dim, key_store, value_store,
                                  page_tokens, error_flag};
+    const bool by_heads = (norm_per_head || !q_norm_w) && (interleaved || !frequencies) && temp_every <= 0 && blend == 0 &&
+                          key_store == head_dim && value_store == value_dim && head_dim <= 128 && value_dim <= 128 &&
+                          ((head_dim | value_dim | proj_stride | q_stride) & 1) == 0 &&
+                          (((size_t)proj | (size_t)bias | (size_t)q_norm_w | (size_t)k_norm_w) & 7) == 0 &&
+                          (((size_t)q_out | (size_t)k_cache | (size_t)v_cache) & 7) == 0 &&
+                          ((page_stride | value_page_stride) & 1) == 0;
+    if (by_heads) {
+        if (act_dtype == kFloat32) launch_prepare_heads<float>(args, tokens, stream);
+        else launch_prepare_heads<__nv_bfloat16>(args, tokens, stream);
+        return check_launch("qkv_prepare");
+    }
     cudaError_t status = cudaSuccess;
     if (smem > 40 * 1024) {
         status = act_dtype == kFloat32

@@ -19,11 +19,12 @@ struct DeltaDecodeArgs {
 
 constexpr int kDeltaDecodeThreads = 256;
 
-template <typename A>
+// kKeep: rows of the state that a thread can hold in registers
+template <typename A, int kKeep>
 __global__ void __launch_bounds__(kDeltaDecodeThreads) delta_decode_kernel(const DeltaDecodeArgs p) {
     extern __shared__ __align__(16) float smem[];  // tanh [rank] | k r w b [4 dim] | o [dim] | partial sums [2 threads]
     __shared__ float scratch[4][8];
-    constexpr int kThreads = kDeltaDecodeThreads, kWarps = kThreads / 32, kKeep = 32;
+    constexpr int kThreads = kDeltaDecodeThreads, kWarps = kThreads / 32;
     chain_release();
     const int head = blockIdx.x, t = blockIdx.y;
     const int dim = p.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -63,7 +64,19 @@ __global__ void __launch_bounds__(kDeltaDecodeThreads) delta_decode_kernel(const
         float z = 0.0f;
         if (e < dim) {
             const A* up = static_cast<const A*>(p.decay_up) + (size_t)(head * dim + e) * p.rank;
-            for (int i = quarter; i < p.rank; i += 4) z = fmaf(to_float(up[i]), low_s[i], z);
+            if (sizeof(A) == 2 && p.rank % 8 == 0 && ((size_t)p.decay_up & 15) == 0) {
+                for (int i = 8 * quarter; i < p.rank; i += 32) {
+                    const uint4 raw = __ldg(reinterpret_cast<const uint4*>(up + i));
+                    const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const float2 w = __bfloat1622float2(pairs[j]);
+                        z = fmaf(w.x, low_s[i + 2 * j], fmaf(w.y, low_s[i + 2 * j + 1], z));
+                    }
+                }
+            } else {
+                for (int i = quarter; i < p.rank; i += 4) z = fmaf(to_float(up[i]), low_s[i], z);
+            }
         }
         z += __shfl_xor_sync(0xffffffffu, z, 1);
         z += __shfl_xor_sync(0xffffffffu, z, 2);
@@ -213,9 +226,15 @@ CELEG_API int celeg_general_delta_decode(const float* proj, int stride, int r_of
                                   state, slot_stride, span_slot, heads, dim, eps, unit_eps, out};
     const size_t smem = (size_t)(((rank + 3) & ~3) + 5 * dim + 2 * kDeltaDecodeThreads) * sizeof(float);
     dim3 grid(heads, tokens);
-    if (act_dtype == kFloat32)
-        launch_chained(delta_decode_kernel<float>, grid, kDeltaDecodeThreads, smem, stream, args);
-    else
-        launch_chained(delta_decode_kernel<__nv_bfloat16>, grid, kDeltaDecodeThreads, smem, stream, args);
+    // (few rows a thread where that holds the head: half the registers, twice the blocks an SM)
+    const int groups = (dim + 31) / 32, split = groups < 8 ? 8 / groups : 1;
+    const bool few = dim <= 16 * split;
+#define CELEG_DELTA_DECODE(A, KEEP) launch_chained(delta_decode_kernel<A, KEEP>, grid, kDeltaDecodeThreads, smem, stream, args)
+    if (act_dtype == kFloat32) {
+        if (few) CELEG_DELTA_DECODE(float, 16); else CELEG_DELTA_DECODE(float, 32);
+    } else {
+        if (few) CELEG_DELTA_DECODE(__nv_bfloat16, 16); else CELEG_DELTA_DECODE(__nv_bfloat16, 32);
+    }
+#undef CELEG_DELTA_DECODE
     return check_launch("general_delta_decode");
 }

@@ -190,6 +190,9 @@ struct DeltaScanArgs {
 
 constexpr int kDeltaWarps = 4;
 
+// What a chunk costs is mostly shared memory's bandwidth (a number that several lanes read costs as much as several
+// numbers) in two phases that the sums among lanes keep apart. Measured at 32 heads of 64 and 2,048 tokens: 290 us; four
+// elements a lane and twice the lanes a column: 340 us; two multiplications an instruction (fma.rn.f32x2): 290 us.
 template <int L>
 __global__ void __launch_bounds__(kDeltaWarps * 32, 1) delta_scan_kernel(const DeltaScanArgs p) {
     constexpr int C = kDeltaChunk, D = 8 * L;
@@ -259,7 +262,7 @@ __global__ void __launch_bounds__(kDeltaWarps * 32, 1) delta_scan_kernel(const D
             const float* inward = base + D + 2 * C * n;        // pairs (-u.b, u.k), i(i-1) floats before token i's
             const float* vectors = base + delta_vectors_at(D, n);
             float su[C], sq[C];
-    #pragma unroll
+#pragma unroll
             for (int i = 0; i < C; ++i) {
                 if (i < n) {
                     const float4* up = reinterpret_cast<const float4*>(vectors + (4 * i) * D);
@@ -274,49 +277,46 @@ __global__ void __launch_bounds__(kDeltaWarps * 32, 1) delta_scan_kernel(const D
                 }
             }
             // the lanes of a column exchange halves: afterwards a lane has the whole sums of its own kMine tokens
-    #pragma unroll
+#pragma unroll
             for (int b = 0; b < kBits; ++b) {
                 const int half = C >> (b + 1);
                 const bool upper = ((sub >> b) & 1) != 0;
-    #pragma unroll
+#pragma unroll
                 for (int i = 0; i < half; ++i) {
                     const float give_u = upper ? su[i] : su[i + half], give_q = upper ? sq[i] : sq[i + half];
                     su[i] = (upper ? su[i + half] : su[i]) + __shfl_xor_sync(0xffffffffu, give_u, 1 << b);
                     sq[i] = (upper ? sq[i + half] : sq[i]) + __shfl_xor_sync(0xffffffffu, give_q, 1 << b);
                 }
             }
-    #pragma unroll
+#pragma unroll
             for (int offset = C; offset < L; offset <<= 1) {
                 su[0] += __shfl_xor_sync(0xffffffffu, su[0], offset);
                 sq[0] += __shfl_xor_sync(0xffffffffu, sq[0], offset);
             }
             float taken[C];                                        // u_i^T S_(i-1), all tokens in every lane
-    #pragma unroll
+#pragma unroll
             for (int i = 0; i < C; ++i) {
                 int from = 0;                                      // which lane of the column holds token i
-    #pragma unroll
+#pragma unroll
                 for (int b = 0; b < kBits; ++b) from |= ((i >> (2 - b)) & 1) << b;
                 taken[i] = __shfl_sync(0xffffffffu, su[i % kMine], (lane & ~((1 << kBits) - 1)) | from);
             }
-    #pragma unroll
+#pragma unroll
             for (int i = 1; i < C; ++i) {
                 if (i < n) {
                     const float2* line = reinterpret_cast<const float2*>(inward + i * (i - 1));
-                    float written = 0.0f;
-    #pragma unroll
-                    for (int j = 0; j < i; ++j) {
-                        const float2 pair = line[j];
-                        taken[i] = fmaf(pair.x, taken[j], taken[i]);
-                        written = fmaf(pair.y, v[j], written);
-                    }
-                    taken[i] += written;
+                    // (the values' share first: then one product only hangs on the token before)
+#pragma unroll
+                    for (int j = 0; j < i; ++j) taken[i] = fmaf(line[j].y, v[j], taken[i]);
+#pragma unroll
+                    for (int j = 0; j < i; ++j) taken[i] = fmaf(line[j].x, taken[j], taken[i]);
                 }
             }
-    #pragma unroll
+#pragma unroll
             for (int m = 0; m < kMine; ++m) {
                 const int i = first_token + m;
                 float removed = 0.0f, written = sq[m];
-    #pragma unroll
+#pragma unroll
                 for (int j = 0; j < C; ++j) {
                     if (j < n) {
                         const float2 pair = *reinterpret_cast<const float2*>(outward + 2 * (j * C + i));
@@ -331,7 +331,7 @@ __global__ void __launch_bounds__(kDeltaWarps * 32, 1) delta_scan_kernel(const D
             const float4 d0 = dp[sub], d1 = dp[L + sub];
             s[0] *= d0.x; s[1] *= d0.y; s[2] *= d0.z; s[3] *= d0.w;
             s[4] *= d1.x; s[5] *= d1.y; s[6] *= d1.z; s[7] *= d1.w;
-    #pragma unroll
+#pragma unroll
             for (int i = 0; i < C; ++i) {
                 if (i < n) {
                     const float4* kp = reinterpret_cast<const float4*>(vectors + (4 * i + 2) * D);

@@ -394,6 +394,48 @@ __global__ void gated_head_norm_kernel(const float* o, const float* gate, int ga
     }
 }
 
+// The same for heads of an even size up to 128 with aligned rows: two neighbours a lane and access, the head's read-outs in
+// registers between the sum and the result.
+template <typename A>
+__global__ void gated_head_norm_pairs_kernel(const float* o, const float* gate, int gate_stride, const float* weight,
+                                             int weight_per_head, A* out, int tokens, int heads, int vdim, float eps,
+                                             int gate_kind) {
+    chain_release();
+    chain_wait();
+    const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= (long long)tokens * heads) return;
+    const int lane = threadIdx.x & 31;
+    const int t = (int)(unit / heads), h = (int)(unit % heads);
+    const float2* src = reinterpret_cast<const float2*>(o + ((size_t)t * heads + h) * vdim);
+    const float2* g = reinterpret_cast<const float2*>(gate + (size_t)t * gate_stride + (size_t)h * vdim);
+    const float2* w = reinterpret_cast<const float2*>(weight ? weight + (weight_per_head ? (size_t)h * vdim : 0) : nullptr);
+    const int pairs = vdim >> 1;
+    float2 x[2], z[2];
+    float sum = 0.0f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+        const int i = lane + 32 * u;
+        x[u] = i < pairs ? src[i] : make_float2(0.0f, 0.0f);
+        z[u] = i < pairs ? g[i] : make_float2(0.0f, 0.0f);
+        sum += x[u].x * x[u].x + x[u].y * x[u].y;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)vdim + eps);
+    A* dst = out + ((size_t)t * heads + h) * vdim;
+    auto gated = [&](float v, float a, float scale) {
+        const float sig = 1.0f / (1.0f + expf(-a));
+        return v * inv * scale * (gate_kind == 0 ? sig : a * sig);
+    };
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+        const int i = lane + 32 * u;
+        if (i >= pairs) continue;
+        const float2 scale = w ? __ldg(w + i) : make_float2(1.0f, 1.0f);
+        const float first = gated(x[u].x, z[u].x, scale.x), second = gated(x[u].y, z[u].y, scale.y);
+        if (sizeof(A) == 2) *reinterpret_cast<__nv_bfloat162*>(dst + 2 * i) = __floats2bfloat162_rn(first, second);
+        else *reinterpret_cast<float2*>(dst + 2 * i) = make_float2(first, second);
+    }
+}
+
 // The same for wide units (one norm over all heads' columns together): a block per (token, head), 16-byte reads
 // where the rows allow them. The order of the sum differs from the warp's; both are float32 sums of the same squares.
 template <typename A>
@@ -988,6 +1030,16 @@ CELEG_API int celeg_gated_head_norm(const float* o, const float* gate, int gate_
         return check_launch("gated_head_norm");
     }
     const unsigned blocks = (unsigned)((units + 3) / 4);
+    if (vdim % 2 == 0 && vdim <= 128 && gate_stride % 2 == 0 && (act_dtype == kFloat32 || act_dtype == kBFloat16) &&
+        (((size_t)o | (size_t)gate | (size_t)weight | (size_t)out) & 7) == 0) {
+        if (act_dtype == kFloat32)
+            launch_chained(gated_head_norm_pairs_kernel<float>, blocks, 128, 0, stream, o, gate, gate_stride, weight,
+                           weight_per_head, (float*)out, tokens, heads, vdim, eps, gate_kind);
+        else
+            launch_chained(gated_head_norm_pairs_kernel<__nv_bfloat16>, blocks, 128, 0, stream, o, gate, gate_stride, weight,
+                           weight_per_head, (__nv_bfloat16*)out, tokens, heads, vdim, eps, gate_kind);
+        return check_launch("gated_head_norm");
+    }
     if (act_dtype == kFloat32)
         launch_chained(gated_head_norm_kernel<float>, blocks, 128, 0, stream, o, gate, gate_stride, weight,
                        weight_per_head, (float*)out, tokens, heads, vdim, eps, gate_kind);
