@@ -207,19 +207,7 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
     const int half = p.frequencies ? p.rotary_dim >> 1 : 0;
     const int q_width = p.q_heads * p.head_dim, qk_width = q_width + p.kv_heads * p.head_dim;
     const float* row = p.proj + (size_t)t * p.proj_stride;
-    if (page < 0 && threadIdx.x == 0) atomicExch(p.error_flag, 2);
     float c[E], s[E];
-#pragma unroll
-    for (int x = 0; x < E; ++x) {
-        c[x] = 1.0f;
-        s[x] = 0.0f;
-        const int pair = lane + 32 * x;
-        if (pair < half) {
-            sincosf((float)pos * p.frequencies[pair], &s[x], &c[x]);
-            c[x] *= p.magnitude;
-            s[x] *= p.magnitude;
-        }
-    }
     const int units = p.q_heads + 2 * p.kv_heads;
     for (int base = warp; base < units; base += kAhead * warps) {
         float2 v[kAhead][E];
@@ -239,6 +227,19 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
                         v[a][x].x += b.x;
                         v[a][x].y += b.y;
                     }
+                }
+            }
+        }
+        if (base == warp) {                                // (the angles, while the first heads are on their way)
+#pragma unroll
+            for (int x = 0; x < E; ++x) {
+                c[x] = 1.0f;
+                s[x] = 0.0f;
+                const int pair = lane + 32 * x;
+                if (pair < half) {
+                    sincosf((float)pos * p.frequencies[pair], &s[x], &c[x]);
+                    c[x] *= p.magnitude;
+                    s[x] *= p.magnitude;
                 }
             }
         }
@@ -281,6 +282,7 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
             }
         }
     }
+    if (page < 0 && threadIdx.x == 0) atomicExch(p.error_flag, 2);
 }
 
 template <typename A>
