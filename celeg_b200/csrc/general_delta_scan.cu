@@ -48,7 +48,7 @@ struct DeltaVectorsArgs {
     const float* w0; const float* a_bias;
     const int* token_span; const int* span_begin;
     float* records;
-    int tokens, heads, dim, padded;
+    int tokens, heads, dim;
     float unit_eps;
 };
 
@@ -423,7 +423,7 @@ CELEG_API int celeg_general_delta_scan(const float* proj, int stride, int r_off,
     if (tokens == 0 || spans == 0) return 0;
     const int padded = delta_padded(dim);
     const DeltaVectorsArgs first = {proj, stride, r_off, k_off, a_off, z, z_stride, w0, a_bias, token_span, span_begin, records,
-                                    tokens, heads, dim, padded, unit_eps};
+                                    tokens, heads, dim, unit_eps};
     const DeltaScanArgs p = {records, proj + v_off, stride, out, state, slot_stride, span_begin, span_slot, tokens, heads, dim,
                              error_flag};
     switch (padded) {

@@ -681,7 +681,7 @@ def large(tmp_path_factory):
     """Four layers 1,024 wide: sixteen recurrent heads of 64 with a decay of rank 64 and 32 experts of 512; sixteen query
     heads of 64 on four key heads; a layer that reads those keys and values; four recurrent heads of 128. The sizes at which
     the grouped tensor-core product, the tcgen05 prompt attention and the split-key decoding are what runs."""
-    rot = km.rotation(250000.0, 32, factor=4.0, original=256, fast=32.0, slow=1.0)
+    rot = km.rotation(300000.0, 32, factor=4.0, original=256, fast=32.0, slow=1.0)
     raw = km.config(4096, 1024, [
         km.with_mlp(km.delta(16, 64, 64), km.moe(32, 4, 512)),
         km.with_mlp(km.attention(16, 4, 64, 64, rot), km.moe(16, 2, 384, limit=2.0)),
