@@ -21,6 +21,9 @@ from .liverax_arch import build_liverax_spec
 from .kodupel import KodupelConfig
 from . import kodupel_arch as _kodupel_arch  # registers "Kodupel"
 from .kodupel_arch import build_kodupel_spec
+from .fovezen import FovezenConfig
+from . import fovezen_arch as _fovezen_arch  # registers "Fovezen"
+from .fovezen_arch import build_fovezen_spec
 
 __all__ = [
     "Architecture", "ConfigError", "UnknownArchitectureError", "ExecutionEntry", "LayerSpec",
@@ -29,4 +32,5 @@ __all__ = [
     "FULL_ATTENTION", "Lfm2Config", "build_lfm2_spec", "RamosunConfig", "build_ramosun_spec",
     "KedesunConfig", "build_kedesun_spec", "NaselornConfig", "build_naselorn_spec",
     "LiveraxConfig", "build_liverax_spec", "KodupelConfig", "build_kodupel_spec",
+    "FovezenConfig", "build_fovezen_spec",
 ]

@@ -49,6 +49,7 @@ struct DecodeParams {
     const float* sinks;            // [q_heads] or null: a score per head that enters the denominator once (no key, no value)
     const float* distance_bias;    // [q_heads, distance_last + 1] or null: added to the scaled score by distance back
     int distance_last;
+    float cap_in, cap_log2;        // softly capped scores: cap_log2 tanh(cap_in * raw score), scale / cap and cap * log2(e); 0: none
     // Optional: the q/k post-processing of the step's own token done here instead of by a kernel of its
     // own. Then q (and the k and v behind it in the same rows: [q heads | k heads | v heads]) is the raw
     // projection; an item normalises and rotates its query heads itself, and the item whose keys include
@@ -337,7 +338,8 @@ __device__ __forceinline__ void attention_decode_item(const DecodeParams& p, con
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = tile_begin + nt * 8 + c2 + (e & 1);
-                float v = key < end ? s[nt][e] * scale_log2 : -INFINITY;
+                float v = key < end ? (p.cap_log2 > 0.0f ? p.cap_log2 * quick_tanh(s[nt][e] * p.cap_in) : s[nt][e] * scale_log2)
+                                    : -INFINITY;
                 if (p.distance_bias && key < end) {
                     // a learned number per (head, distance back to the key) joins the scaled score, in units of log2
                     const int row = min(g + (e >> 1) * 8, group - 1);      // (rows past the group are never stored)
@@ -726,7 +728,8 @@ __device__ __forceinline__ void attention_decode_item_solo(const DecodeParams& p
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = tile_begin + nt * 8 + c2 + (e & 1);
-                float v = key < end ? s[nt][e] * scale_log2 : -INFINITY;
+                float v = key < end ? (p.cap_log2 > 0.0f ? p.cap_log2 * quick_tanh(s[nt][e] * p.cap_in) : s[nt][e] * scale_log2)
+                                    : -INFINITY;
                 if (p.distance_bias && key < end) {
                     // a learned number per (head, distance back to the key) joins the scaled score, in units of log2
                     const int row = min(g + (e >> 1) * 8, group - 1);      // (rows past the group are never stored)

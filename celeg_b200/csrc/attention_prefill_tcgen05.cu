@@ -61,6 +61,9 @@ struct FaParams {
     const float* distance_bias;
     int distance_last;
     float bias_factor;
+    // softly capped scores: cap_out tanh(cap_in * raw score), scale / cap and cap / scale (so that the result is again in
+    // the unit of the raw scores); 0: none
+    float cap_in, cap_out;
     int* error_flag;
 };
 
@@ -268,6 +271,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                         sc[32 + j] = __uint_as_float(hi[j]);
                     }
                 }
+                if (p.cap_out > 0.0f) {
+#pragma unroll
+                    for (int j = 0; j < kFaN; ++j) sc[j] = p.cap_out * quick_tanh(sc[j] * p.cap_in);
+                }
                 if (p.distance_bias) {
                     const float* bias = p.distance_bias + (size_t)h * (p.distance_last + 1);
                     const int back = qpos - key_base;               // key key_base + j lies back - j positions back
@@ -424,9 +431,9 @@ CELEG_API int celeg_attention_prefill_tcgen05(const void* q, int q_row_stride, i
                                               int tokens, int spans, int tile_count, int q_heads, int kv_heads,
                                               int head_dim, int page_tokens, int window, float scale,
                                               const float* sinks, const float* distance_bias, int distance_last,
-                                              int* error_flag, cudaStream_t stream) {
-    CELEG_REQUIRE(!distance_bias || scale > 0.0f, "attention_prefill_tcgen05: score biases need a positive scale, got %g",
-                  scale);
+                                              float softcap, int* error_flag, cudaStream_t stream) {
+    CELEG_REQUIRE((!distance_bias && softcap <= 0.0f) || scale > 0.0f,
+                  "attention_prefill_tcgen05: score biases and capped scores need a positive scale, got %g", scale);
     CELEG_REQUIRE(celeg_attention_prefill_tcgen05_supported(q_heads, kv_heads, head_dim, page_tokens),
                   "attention_prefill_tcgen05: head_dim=%d page_tokens=%d q_heads=%d kv_heads=%d are not taken here",
                   head_dim, page_tokens, q_heads, kv_heads);
@@ -457,6 +464,8 @@ CELEG_API int celeg_attention_prefill_tcgen05(const void* q, int q_row_stride, i
     p.distance_bias = distance_bias;
     p.distance_last = distance_last;
     p.bias_factor = distance_bias ? 1.0f / scale : 0.0f;
+    p.cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.cap_out = softcap > 0.0f ? softcap / scale : 0.0f;
     p.error_flag = error_flag;
     const cudaError_t status = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel,
                                                     cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kFaSmemBytes);

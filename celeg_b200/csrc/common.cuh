@@ -71,6 +71,14 @@ __device__ __forceinline__ float activate(float z, int kind) {
     return z / (1.0f + expf(-z));
 }
 
+// tanh by one exponential and one quotient, 1 - 2 / (1 + e^(2x)): within 3e-7 of it, whatever x is. For scores that are
+// capped softly on the bfloat16 path, where a number of the order of the cap meets an exponential.
+__device__ __forceinline__ float quick_tanh(float x) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
+    return 1.0f - __fdividef(2.0f, 1.0f + e);
+}
+
 // What a gated linear unit makes of a gate and an up value: activate(g) * u, or with kClampedSilu the clamped form
 // g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).
 constexpr int kClampedSilu = 6;

@@ -585,11 +585,12 @@ using namespace celeg_b200;
 
 // c[m, n] = a[m, k] * b[n, k]^T in bfloat16 with float32 accumulation on tcgen05 tensor cores.
 // epilogue 0: c bfloat16; 1: c float32; 2: b holds n gate rows then n up rows, c bfloat16 [m, n] =
-// silu(a gate^T) * (a up^T) (16 + kind: the same with activate(., kind) on the gate); 3, 4, 5: c bfloat16 = act(a b^T) with the exact GELU, the tanh GELU, SiLU. k, lda and ldb must be multiples of 8 (16-byte rows for TMA); operands
+// silu(a gate^T) * (a up^T) (16 + kind: the same with activate(., kind) on the gate, or the clamped form with its constants limit, slope, shift); 3, 4, 5: c bfloat16 = act(a b^T) with the exact GELU, the tanh GELU, SiLU. k, lda and ldb must be multiples of 8 (16-byte rows for TMA); operands
 // 16-byte aligned. error_flag (device int) receives a code if a bounded wait inside the kernel ran out.
 // forced_variant: -1 = the kernel is chosen from the shape, 0..3 = that one (for measurements).
 CELEG_API int celeg_gemm_tcgen05(const void* a, int lda, const void* b, int ldb, void* c, int ldc, int m, int n, int k,
-                                 int epilogue, int* error_flag, int forced_variant, cudaStream_t stream) {
+                                 int epilogue, float limit, float slope, float shift, int* error_flag, int forced_variant,
+                                 cudaStream_t stream) {
     CELEG_REQUIRE(m > 0 && n > 0 && k > 0, "gemm_tcgen05: invalid sizes m=%d n=%d k=%d", m, n, k);
     CELEG_REQUIRE(k % 8 == 0 && lda % 8 == 0 && ldb % 8 == 0 && lda >= k && ldb >= k,
                   "gemm_tcgen05: k=%d, lda=%d and ldb=%d must be multiples of 8 and cover k", k, lda, ldb);
@@ -597,7 +598,7 @@ CELEG_API int celeg_gemm_tcgen05(const void* a, int lda, const void* b, int ldb,
     CELEG_REQUIRE(ldc >= n && error_flag != nullptr, "gemm_tcgen05: ldc=%d is smaller than n=%d, or no error flag", ldc, n);
     // 16 + kind: the gated form with activate(gate, kind) in place of SiLU
     int gate_activation = kSilu;
-    if (epilogue >= 16 && epilogue <= 16 + kRelu) {
+    if ((epilogue >= 16 && epilogue <= 16 + kRelu) || epilogue == 16 + kClampedSilu) {
         gate_activation = epilogue - 16;
         epilogue = kTcSwiGlu;
     }
@@ -615,7 +616,7 @@ CELEG_API int celeg_gemm_tcgen05(const void* a, int lda, const void* b, int ldb,
     if (!tensor_map_for(b, b_rows, k, ldb, epilogue == kTcSwiGlu ? bn / 2 : bn, &map_b)) return -3;
     TcGemmParams p{m, n, k, c, ldc, error_flag,
                    epilogue >= kTcActivation ? epilogue - kTcActivation : (epilogue == kTcSwiGlu ? gate_activation : 0),
-                   nullptr, 0, {0.0f, 0.0f, 0.0f}};
+                   nullptr, 0, {limit, slope, shift}};
     if (epilogue > kTcActivation) epilogue = kTcActivation;
 #define CELEG_TC_DISPATCH(BN, STAGES)                                                        \
     switch (epilogue) {                                                                      \

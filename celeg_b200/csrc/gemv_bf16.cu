@@ -34,7 +34,8 @@ constexpr int kGemvMaxConvTaps = 16;
 
 enum GemvMode : int { kGemvStoreBf16 = 0, kGemvStoreF32 = 1, kGemvAddResidual = 2, kGemvSwiGlu = 3, kGemvConv = 4,
                       kGemvActivation = 5 };     // y bfloat16 = act(x w^T); which activation travels in the `taps` argument
-// (kGemvSwiglu: `taps` = 1 + a code of activate() names another function of the gate than SiLU; 0: SiLU)
+// (kGemvSwiglu: `taps` = 1 + a code of activate(), or of the clamped form, names another function of the gate than SiLU;
+// 0: SiLU)
 
 struct GemvConvArgs {
     const float* conv_w;         // [channels, taps]
@@ -42,6 +43,7 @@ struct GemvConvArgs {
     float* state;                // this layer's state inside slot 0: [taps-1][channels] per slot
     long long slot_stride;
     const int* span_slot;        // state slot of row i (row i is the single token of span i)
+    GateConstants gate;          // of kClampedSilu (SwiGLU mode)
 };
 
 // The norm between two products, split over them. The product that ends a part adds its result to
@@ -362,7 +364,7 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
             const float gate = __bfloat162float(__float2bfloat16_rn(sum[0]));
             const float up = __bfloat162float(__float2bfloat16_rn(sum[WT - 1]));
             reinterpret_cast<__nv_bfloat16*>(y)[(size_t)out_row * ldy + out_col] =
-                __float2bfloat16_rn((conv.taps > 0 ? activate(gate, conv.taps - 1) : gate / (1.0f + expf(-gate))) * up);
+                __float2bfloat16_rn(conv.taps > 0 ? gated_value(gate, up, conv.taps - 1, conv.gate) : gate / (1.0f + expf(-gate)) * up);
         }
     }
     if (MODE == kGemvAddResidual && norm.next_w) {
@@ -425,6 +427,7 @@ static int launch_gemv(int mode, const __nv_bfloat16* x, int ldx, const __nv_bfl
     return -1;
 }
 
+static thread_local GateConstants g_gemv_gate = {0.0f, 0.0f, 0.0f};      // of the next product with a clamped gate
 static int g_gemv_warps = 0;      // 0: chosen from the shape; 8, 16 or 32: forced (for measurements)
 
 }  // namespace celeg_b200
@@ -432,6 +435,12 @@ static int g_gemv_warps = 0;      // 0: chosen from the shape; 8, 16 or 32: forc
 using namespace celeg_b200;
 
 CELEG_API void celeg_gemv_set_warps(int warps) { g_gemv_warps = warps; }
+
+// The constants of the clamped gated form (see gated_value) for the products of this thread that name it.
+CELEG_API int celeg_gemv_gate_constants(float limit, float slope, float shift) {
+    g_gemv_gate = {limit, slope, shift};
+    return 0;
+}
 
 // A hint for the next celeg_gemv_bf16* launch only: `bytes` of device memory at `ptr` (the weights that the
 // product after it will read) are asked into the L2 by that launch's blocks. The memory must stay
@@ -468,7 +477,7 @@ static int gemv_checked(const void* x, int ldx, const void* w, int ldw, void* y,
     g_gemv_launch_ahead = ahead;
     const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
     const __nv_bfloat16* wp = (const __nv_bfloat16*)w;
-    GemvConvArgs conv = {conv_w, taps, state, slot_stride, span_slot};
+    GemvConvArgs conv = {conv_w, taps, state, slot_stride, span_slot, g_gemv_gate};
     // blocks = n/16. A narrow matrix has fewer blocks than SMs; then only more warps per block put
     // enough loads in flight (each warp keeps 4 x 1 KiB of weights in flight, HBM needs some 50 KiB
     // per SM). Measured on B200 at 8 rows: 2048x8192 11.2 us with 8 warps, 8.7 us with 32; 2048x2048

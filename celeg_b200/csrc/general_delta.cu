@@ -179,7 +179,7 @@ __global__ void __launch_bounds__(kDeltaDecodeThreads) delta_decode_kernel(const
     }
 }
 
-// out[t, c] = act(x[t, c]) of float32 columns that lie in wider rows, rounded once
+// out[t, c] = act(x[t, c]) of float32 columns that lie in wider rows, rounded once (kind -1: no function)
 template <typename A>
 __global__ void activation_cast_kernel(const float* x, long long stride, A* out, int tokens, int columns, int kind) {
     chain_release();
@@ -187,7 +187,7 @@ __global__ void activation_cast_kernel(const float* x, long long stride, A* out,
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)tokens * columns) return;
     const int t = (int)(i / columns), c = (int)(i % columns);
-    out[i] = from_float<A>(activate(x[(size_t)t * stride + c], kind));
+    out[i] = from_float<A>(kind < 0 ? x[(size_t)t * stride + c] : activate(x[(size_t)t * stride + c], kind));
 }
 
 }  // namespace celeg_b200
@@ -196,7 +196,7 @@ using namespace celeg_b200;
 
 CELEG_API int celeg_activation_cast(const float* x, long long stride, void* out, int tokens, int columns, int kind,
                                     int act_dtype, cudaStream_t stream) {
-    CELEG_REQUIRE(tokens >= 0 && columns > 0 && stride >= columns && kind >= 0 && kind <= kTanh,
+    CELEG_REQUIRE(tokens >= 0 && columns > 0 && stride >= columns && kind >= -1 && kind <= kTanh,
                   "activation_cast: invalid sizes tokens=%d columns=%d stride=%lld kind=%d", tokens, columns, stride, kind);
     CELEG_REQUIRE(act_dtype == kFloat32 || act_dtype == kBFloat16, "activation_cast: unknown dtype code %d", act_dtype);
     if (tokens == 0) return 0;

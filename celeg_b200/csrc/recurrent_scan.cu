@@ -367,8 +367,14 @@ __global__ void carried_inputs_update_kernel(const float* proj, int stride, floa
         if (r < taps - 1) mine[(size_t)r * channels + c] = keep[r];
 }
 
-// One warp per (token, head): o / sqrt(mean(o^2) + eps) * w * act(gate), act = sigmoid (0) or SiLU (1);
-// w is [heads * vdim] or, shared by the heads, [vdim].
+// One warp per (token, head): o / sqrt(mean(o^2) + eps) * w * act(gate), act = sigmoid (0) or SiLU (1); with 2 or 3 the
+// sigmoid or SiLU is applied before the norm, x / sqrt(mean(x^2) + eps) * w of x = o * act(gate). w is [heads * vdim] or,
+// shared by the heads, [vdim].
+__device__ __forceinline__ float output_gate(float z, int kind) {
+    const float sig = 1.0f / (1.0f + expf(-z));
+    return (kind & 1) ? z * sig : sig;
+}
+
 template <typename A>
 __global__ void gated_head_norm_kernel(const float* o, const float* gate, int gate_stride, const float* weight,
                                        int weight_per_head, A* out, int tokens, int heads, int vdim, float eps,
@@ -380,18 +386,18 @@ __global__ void gated_head_norm_kernel(const float* o, const float* gate, int ga
     const int lane = threadIdx.x & 31;
     const int t = (int)(unit / heads), h = (int)(unit % heads);
     const float* src = o + ((size_t)t * heads + h) * vdim;
-    float sum = 0.0f;
-    for (int i = lane; i < vdim; i += 32) sum += src[i] * src[i];
-    sum = warp_sum(sum);
-    const float inv = 1.0f / sqrtf(sum / (float)vdim + eps);
     const float* w = weight ? weight + (weight_per_head ? (size_t)h * vdim : 0) : nullptr;     // (null: no weight)
     const float* g = gate + (size_t)t * gate_stride + (size_t)h * vdim;
-    A* dst = out + ((size_t)t * heads + h) * vdim;
+    float sum = 0.0f;
     for (int i = lane; i < vdim; i += 32) {
-        const float z = g[i];
-        const float sig = 1.0f / (1.0f + expf(-z));
-        dst[i] = from_float<A>(src[i] * inv * (w ? w[i] : 1.0f) * (gate_kind == 0 ? sig : z * sig));
+        const float x = gate_kind >= 2 ? src[i] * output_gate(g[i], gate_kind) : src[i];
+        sum += x * x;
     }
+    sum = warp_sum(sum);
+    const float inv = 1.0f / sqrtf(sum / (float)vdim + eps);
+    A* dst = out + ((size_t)t * heads + h) * vdim;
+    for (int i = lane; i < vdim; i += 32)
+        dst[i] = from_float<A>(src[i] * inv * (w ? w[i] : 1.0f) * output_gate(g[i], gate_kind));
 }
 
 // The same for heads of an even size up to 128 with aligned rows: two neighbours a lane and access, the head's read-outs in
@@ -417,13 +423,16 @@ __global__ void gated_head_norm_pairs_kernel(const float* o, const float* gate, 
         const int i = lane + 32 * u;
         x[u] = i < pairs ? src[i] : make_float2(0.0f, 0.0f);
         z[u] = i < pairs ? g[i] : make_float2(0.0f, 0.0f);
+        if (gate_kind >= 2) {
+            x[u].x *= output_gate(z[u].x, gate_kind);
+            x[u].y *= output_gate(z[u].y, gate_kind);
+        }
         sum += x[u].x * x[u].x + x[u].y * x[u].y;
     }
     const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)vdim + eps);
     A* dst = out + ((size_t)t * heads + h) * vdim;
     auto gated = [&](float v, float a, float scale) {
-        const float sig = 1.0f / (1.0f + expf(-a));
-        return v * inv * scale * (gate_kind == 0 ? sig : a * sig);
+        return v * inv * scale * (gate_kind >= 2 ? 1.0f : output_gate(a, gate_kind));
     };
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -454,11 +463,19 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const float* o, con
     float sum = 0.0f;
     if (vectors) {
         for (int i = threadIdx.x * 4; i < vdim; i += blockDim.x * 4) {
-            const float4 v = *reinterpret_cast<const float4*>(src + i);
+            float4 v = *reinterpret_cast<const float4*>(src + i);
+            if (gate_kind >= 2) {
+                const float4 z = *reinterpret_cast<const float4*>(g + i);
+                v.x *= output_gate(z.x, gate_kind); v.y *= output_gate(z.y, gate_kind);
+                v.z *= output_gate(z.z, gate_kind); v.w *= output_gate(z.w, gate_kind);
+            }
             sum += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
     } else {
-        for (int i = threadIdx.x; i < vdim; i += blockDim.x) sum += src[i] * src[i];
+        for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
+            const float x = gate_kind >= 2 ? src[i] * output_gate(g[i], gate_kind) : src[i];
+            sum += x * x;
+        }
     }
     sum = warp_sum(sum);
     if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum;
@@ -466,10 +483,7 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const float* o, con
     sum = 0.0f;
     for (int k = 0; k < (int)(blockDim.x >> 5); ++k) sum += partial[k];      // (every thread adds in the same order)
     const float inv = 1.0f / sqrtf(sum / (float)vdim + eps);
-    auto one = [&](float x, float z, float scale) {
-        const float sig = 1.0f / (1.0f + expf(-z));
-        return x * inv * scale * (gate_kind == 0 ? sig : z * sig);
-    };
+    auto one = [&](float x, float z, float scale) { return x * inv * scale * output_gate(z, gate_kind); };
     if (vectors) {
         for (int i = threadIdx.x * 4; i < vdim; i += blockDim.x * 4) {
             const float4 v = *reinterpret_cast<const float4*>(src + i);
@@ -1011,7 +1025,7 @@ CELEG_API int celeg_delta_prepare(const float* proj, int stride, const float* ke
 CELEG_API int celeg_gated_head_norm(const float* o, const float* gate, int gate_stride, const float* weight,
                                     int weight_per_head, void* out, int tokens, int heads, int vdim, float eps,
                                     int gate_kind, int act_dtype, cudaStream_t stream) {
-    CELEG_REQUIRE(tokens >= 0 && heads > 0 && vdim > 0 && eps > 0.0f && (gate_kind == 0 || gate_kind == 1),
+    CELEG_REQUIRE(tokens >= 0 && heads > 0 && vdim > 0 && eps > 0.0f && (gate_kind >= 0 && gate_kind <= 3),
                   "gated_head_norm: invalid sizes tokens=%d heads=%d vdim=%d eps=%g gate=%d", tokens, heads, vdim, eps,
                   gate_kind);
     if (tokens == 0) return 0;

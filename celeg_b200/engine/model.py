@@ -189,6 +189,7 @@ class Model:
         rt = self.rt
         stream = self.stream
         stream.begin()
+        step.extras.clear()                    # (what parts of an earlier run left for later ones: it must be made anew)
         blocks = [self.layers[entry.layer].block for entry in self.order]
         firsts = [block.first_norm(step) if hasattr(block, "first_norm") else None for block in blocks]
         head_norm = self.output.next_norm(step, n_logits) if hasattr(self.output, "next_norm") else None

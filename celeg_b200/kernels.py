@@ -46,7 +46,7 @@ _SIGNATURES = {
                                  c_int, c_void_p, c_int, c_void_p],
     "celeg_attention_generic": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int,
                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
+                                c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p],
     "celeg_qkv_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_float, c_void_p, c_int,
                           c_int, c_float, c_float, c_int, c_int,
                           c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
@@ -96,13 +96,14 @@ _SIGNATURES = {
     "celeg_attention_decode_resident_blocks": [c_int],
     "celeg_attention_prefill": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                                 c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p],
     "celeg_attention_prefill_tcgen05": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                         c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                        c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                        c_float, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p],
     "celeg_attention_decode_biased": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-                                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p],
+    "celeg_gemv_gate_constants": [c_float, c_float, c_float],
     "celeg_gemv_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                         c_void_p, c_longlong, c_void_p, c_void_p],
     "celeg_gemv_prefetch_next": [c_void_p, c_longlong],
@@ -111,8 +112,8 @@ _SIGNATURES = {
                                    c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
     "celeg_embedding_split_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
                                    c_void_p, c_int, c_void_p],
-    "celeg_gemm_tcgen05": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                           c_int, c_void_p],
+    "celeg_gemm_tcgen05": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                           c_float, c_void_p, c_int, c_void_p],
     "celeg_swiglu": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "celeg_gemm_f32": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "celeg_sample": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -165,6 +166,26 @@ _SIGNATURES = {
                              c_int, c_int, c_int, c_int, c_void_p],
     "celeg_expert_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int,
                           c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
+    "celeg_hyper_connect": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_longlong, c_void_p, c_longlong, c_void_p,
+                            c_void_p, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int,
+                            c_void_p, c_int, c_int, c_void_p],
+    "celeg_normed_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+    "celeg_channel_conv": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                           c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_chunk_tokens": [],
+    "celeg_chunk_plan": [c_void_p, c_int, c_int, c_void_p, c_void_p],
+    "celeg_channel_decay_scan": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_float,
+                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
+                                 c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_scalar_decay_scan": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
+                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "celeg_channel_decay_decode": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int,
+                                   c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int,
+                                   c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+    "celeg_scalar_decay_decode": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                                  c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                  c_void_p],
     "celeg_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p],
 }
@@ -380,12 +401,14 @@ def attention_generic(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_c
                       block_table: torch.Tensor, tokens: int, q_heads: int, kv_heads: int, head_dim: int,
                       page_tokens: int, window: Optional[int], scale: float, error_flag: torch.Tensor,
                       sinks: Optional[torch.Tensor] = None, value_dim: Optional[int] = None,
-                      chunk: Optional[int] = None, distance_bias: Optional[torch.Tensor] = None) -> None:
+                      chunk: Optional[int] = None, distance_bias: Optional[torch.Tensor] = None,
+                      softcap: Optional[float] = None) -> None:
     """``sinks``: float32 [q_heads] or None; a head's sink is a score that enters the denominator of each of its
     rows once, unscaled, without key or value. ``value_dim``: the values' size when it is not the keys' (``out`` is
     then [tokens, q_heads * value_dim]). ``chunk``: a query reads only the keys of its own chunk of that many
     positions, counted from position 0 (no window then). ``distance_bias``: float32 [q_heads, n + 1] or None; entry
-    [h, min(distance, n)] is added to head h's scaled score of a key ``distance`` positions back."""
+    [h, min(distance, n)] is added to head h's scaled score of a key ``distance`` positions back. ``softcap``: scaled
+    scores s become softcap tanh(s / softcap) first."""
     if sinks is not None:
         _need(sinks, torch.float32, "sinks")
     bias_ptr, bias_last = _distance_bias(distance_bias, q_heads)
@@ -393,8 +416,8 @@ def attention_generic(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_c
         _ptr(q), q_row_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.stride(0), v_cache.stride(0),
         int(value_dim or 0), int(chunk or 0), _ptr(positions),
         _ptr(token_span), _ptr(block_table), block_table.stride(0), tokens, q_heads, kv_heads, head_dim,
-        page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, _ptr(error_flag), dtype_code(q.dtype),
-        _stream()))
+        page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, float(softcap or 0.0), _ptr(error_flag),
+        dtype_code(q.dtype), _stream()))
 
 
 def _distance_bias(table: Optional[torch.Tensor], q_heads: int) -> Tuple[Optional[int], int]:
@@ -510,16 +533,16 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_ca
                      page_tokens: int, window: Optional[int], scale: float, chunk: int, max_splits: int,
                      partial_o: torch.Tensor, partial_ml: torch.Tensor, counters: torch.Tensor,
                      error_flag: torch.Tensor, sinks: Optional[torch.Tensor] = None,
-                     distance_bias: Optional[torch.Tensor] = None) -> None:
+                     distance_bias: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
     """One query token per row, keys split into chunks of ``chunk``; scratch: partial_o float32
     [tokens*q_heads*max_splits*head_dim], partial_ml float32 [tokens*q_heads*max_splits*2],
     counters int32 [tokens*kv_heads] (zero before the first call, left zero by every call).
-    ``sinks``: as for :func:`attention_generic`. ``window`` = -c (negative) stands for a chunked mask: a query reads the
+    ``sinks``, ``softcap``: as for :func:`attention_generic`. ``window`` = -c (negative) stands for a chunked mask: a query reads the
     keys of its own chunk of c positions, chunks counted from position 0; the prompt kernels read it the same way."""
     assert partial_o.numel() >= tokens * q_heads * max_splits * head_dim
     assert partial_ml.numel() >= tokens * q_heads * max_splits * 2
     assert counters.numel() >= tokens * kv_heads
-    if distance_bias is not None:
+    if distance_bias is not None or softcap:
         if sinks is not None:
             _need(sinks, torch.float32, "sinks")
         bias_ptr, bias_last = _distance_bias(distance_bias, q_heads)
@@ -527,7 +550,7 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_ca
             _ptr(q), q_row_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.stride(0), _ptr(positions),
             _ptr(token_span), _ptr(block_table), block_table.stride(0), tokens, q_heads, kv_heads, head_dim,
             page_tokens, int(window or 0), scale, chunk, max_splits, _ptr(partial_o), _ptr(partial_ml),
-            _ptr(counters), _ptr(error_flag), _ptr(sinks), bias_ptr, bias_last, _stream()))
+            _ptr(counters), _ptr(error_flag), _ptr(sinks), bias_ptr, bias_last, float(softcap or 0.0), _stream()))
         return
     if sinks is not None:
         _need(sinks, torch.float32, "sinks")
@@ -571,14 +594,15 @@ def attention_prefill(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_c
                       block_table: torch.Tensor, tokens: int, spans: int, q_heads: int, kv_heads: int,
                       head_dim: int, page_tokens: int, window: Optional[int], scale: float,
                       error_flag: torch.Tensor, sinks: Optional[torch.Tensor] = None,
-                      distance_bias: Optional[torch.Tensor] = None) -> None:
+                      distance_bias: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
     if sinks is not None:
         _need(sinks, torch.float32, "sinks")
     bias_ptr, bias_last = _distance_bias(distance_bias, q_heads)
     _check(library().celeg_attention_prefill(
         _ptr(q), q_row_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.stride(0), _ptr(positions),
         _ptr(span_begin), _ptr(block_table), block_table.stride(0), tokens, spans, q_heads, kv_heads, head_dim,
-        page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, _ptr(error_flag), _stream()))
+        page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, float(softcap or 0.0), _ptr(error_flag),
+        _stream()))
 
 
 def attention_prefill_tcgen05_supported(q_heads: int, kv_heads: int, head_dim: int, page_tokens: int,
@@ -593,9 +617,9 @@ def attention_prefill_tcgen05(q: torch.Tensor, q_row_stride: int, out: torch.Ten
                               block_table: torch.Tensor, tokens: int, spans: int, tile_count: int, q_heads: int,
                               kv_heads: int, head_dim: int, page_tokens: int, window: Optional[int], scale: float,
                               error_flag: torch.Tensor, sinks: Optional[torch.Tensor] = None,
-                              distance_bias: Optional[torch.Tensor] = None) -> None:
+                              distance_bias: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
     """Prompt-portion attention on tcgen05 (S and O' in tensor memory, Q/K/V by TMA).
-    ``tile_count`` = sum over the spans of ceil(length / 128). ``distance_bias``: as for :func:`attention_generic`."""
+    ``tile_count`` = sum over the spans of ceil(length / 128). ``distance_bias``, ``softcap``: as for :func:`attention_generic`."""
     if not (k_cache.is_contiguous() and v_cache.is_contiguous()):
         raise KernelLibraryError("attention_prefill_tcgen05 needs contiguous cache layers")
     if sinks is not None:
@@ -604,7 +628,8 @@ def attention_prefill_tcgen05(q: torch.Tensor, q_row_stride: int, out: torch.Ten
     _check(library().celeg_attention_prefill_tcgen05(
         _ptr(q), q_row_stride, q.shape[0], _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(positions),
         _ptr(span_begin), _ptr(block_table), block_table.stride(0), tokens, spans, tile_count, q_heads, kv_heads,
-        head_dim, page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, _ptr(error_flag), _stream()))
+        head_dim, page_tokens, int(window or 0), scale, _ptr(sinks), bias_ptr, bias_last, float(softcap or 0.0),
+        _ptr(error_flag), _stream()))
 
 
 ACT_GELU_ERF, ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED, ACT_RELU, ACT_TANH = 0, 1, 2, 3, 4, 5      # codes of csrc/common.cuh: activate()
@@ -623,11 +648,12 @@ def gemv_bf16(x, w: torch.Tensor, y: torch.Tensor, rows: int, mode: int = GEMV_S
               conv_w: Optional[torch.Tensor] = None, taps: int = 0, state: Optional[torch.Tensor] = None,
               slot_stride: int = 0, span_slot: Optional[torch.Tensor] = None,
               prepare: Optional[SplitNorm] = None, next_weight: Optional[torch.Tensor] = None,
-              ahead: Optional[Tuple[int, int]] = None) -> None:
+              ahead: Optional[Tuple[int, int]] = None,
+              gate_constants: Optional[Tuple[float, float, float]] = None) -> None:
     """y[:rows] = x[:rows] @ w.T for at most 16 rows, streaming w once. mode GEMV_STORE: y bfloat16;
     GEMV_STORE_F32: y float32; GEMV_ADD_RESIDUAL: y float32, accumulated; GEMV_SWIGLU: w is
     [2*inner, k] (gate rows, then up rows) and y bfloat16 [rows, inner] = silu(gate) * up (``taps`` = 1 + ACT_*:
-    that function of the gate instead); GEMV_CONV: w is
+    that function of the gate instead, or 1 + GATE_CLAMPED_SILU with its ``gate_constants``); GEMV_CONV: w is
     [3*channels, k] (B, C, X rows of the short convolution's input projection), y bfloat16
     [rows, channels] = C * conv(B*X) over each request's carried state, which is shifted; row i is the
     single token of request i, whose state slot is span_slot[i]. GEMV_ACTIVATION: y bfloat16 = act(x w^T) with
@@ -641,6 +667,8 @@ def gemv_bf16(x, w: torch.Tensor, y: torch.Tensor, rows: int, mode: int = GEMV_S
     if ahead is not None and ahead[1] > 0:
         if library().celeg_gemv_prefetch_next(ctypes.c_void_p(ahead[0]), ahead[1]) != 0:      # (no launch)
             raise KernelLibraryError(library().celeg_last_error().decode("utf-8", "replace"))
+    if gate_constants is not None:
+        library().celeg_gemv_gate_constants(*gate_constants)      # (no launch)
     blocks = {GEMV_SWIGLU: 2, GEMV_CONV: 3}.get(mode, 1)
     n = w.shape[0] // blocks
     k = w.shape[1]
@@ -681,10 +709,12 @@ def gemm_tcgen05_supported(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, rows: int, epilogue: int,
-                 error_flag: torch.Tensor, variant: int = -1) -> None:
+                 error_flag: torch.Tensor, variant: int = -1,
+                 gate_constants: Tuple[float, float, float] = NO_GATE_CONSTANTS) -> None:
     """y[:rows] = x[:rows] @ w.T on tcgen05 tensor cores (TMA-fed, accumulator in tensor memory).
     TC_STORE: y bfloat16; TC_STORE_F32: y float32; TC_SWIGLU: w is [2*inner, k] (gate rows, then up rows),
-    y bfloat16 [rows, inner] = silu(gate) * up; TC_GATED + kind: the same with another function of the gate.
+    y bfloat16 [rows, inner] = silu(gate) * up; TC_GATED + kind: the same with another function of the gate
+    (GATE_CLAMPED_SILU takes ``gate_constants``).
     ``variant``: -1 lets the library choose the tile shape,
     0..3 force one (128x128 with 6 or 3 stages, 128x256, persistent with two accumulators)."""
     n = w.shape[0] // 2 if epilogue == TC_SWIGLU or epilogue >= TC_GATED else w.shape[0]
@@ -694,7 +724,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, rows: int, e
         raise KernelLibraryError(f"gemm_tcgen05 epilogue {epilogue} writes {want}, got {y.dtype}")
     assert x.shape[-1] == k and y.shape[-1] >= n
     _check(library().celeg_gemm_tcgen05(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(y), y.stride(0), rows, n, k,
-                                        epilogue, _ptr(error_flag), int(variant), _stream()))
+                                        epilogue, *gate_constants, _ptr(error_flag), int(variant), _stream()))
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, tokens: int, inner: int) -> None:
@@ -922,12 +952,14 @@ def delta_prepare(proj: torch.Tensor, kernel: torch.Tensor, carried: torch.Tenso
 
 
 GATE_SIGMOID, GATE_SILU = 0, 1
+GATE_BEFORE_NORM = 2        # added to either: the gate is applied to what is normed
 
 
 def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], weight_per_head: bool,
                     out: torch.Tensor, tokens: int, heads: int, vdim: int, eps: float, gate_kind: int) -> None:
     """out = o / sqrt(mean_head(o^2) + eps) * weight * act(gate) per (token, head); o and gate float32; ``weight``
-    None: no weight."""
+    None: no weight. With GATE_BEFORE_NORM added to ``gate_kind``: out = x / sqrt(mean_head(x^2) + eps) * weight of
+    x = o * act(gate)."""
     assert o.dtype == torch.float32 and gate.dtype == torch.float32 and o.is_contiguous() and gate.stride(-1) == 1
     _check(library().celeg_gated_head_norm(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), int(weight_per_head),
                                            _ptr(out), tokens, heads, vdim, eps, gate_kind, dtype_code(out.dtype),
@@ -949,7 +981,8 @@ def retention_decode_raw(proj: torch.Tensor, offsets: Tuple[int, int, int], deca
 
 # ------------------------------------------------------------------------------- generalised delta rule
 def activation_cast(x: torch.Tensor, out: torch.Tensor, tokens: int, kind: int) -> None:
-    """out[:tokens] = act(x[:tokens]) of float32 columns that lie in wider rows, rounded once to the type of ``out``."""
+    """out[:tokens] = act(x[:tokens]) of float32 columns that lie in wider rows, rounded once to the type of ``out``;
+    ``kind`` -1: no function."""
     assert x.dtype == torch.float32 and x.stride(-1) == 1 and out.is_contiguous() and x.shape[-1] == out.shape[-1]
     _check(library().celeg_activation_cast(_ptr(x), x.stride(0), _ptr(out), tokens, out.shape[-1], kind,
                                            dtype_code(out.dtype), _stream()))
@@ -1225,3 +1258,142 @@ def moe_combine(expert_out: torch.Tensor, place_of_pair: Optional[torch.Tensor],
     _check(library().celeg_moe_combine(_ptr(expert_out), expert_out.stride(0), _ptr(place_of_pair), _ptr(weights),
                                        _ptr(shared), _ptr(shared_gate), _ptr(y), tokens, width, top,
                                        dtype_code(y.dtype), _stream()))
+
+
+# ------------------------------------ several residual streams, channel convolutions, token-dependent decays
+def hyper_connect(streams: torch.Tensor, count: int, out: torch.Tensor, rows: int, width: int, *,
+                  single: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, y2: Optional[torch.Tensor] = None,
+                  y_norms: Optional[Tuple[torch.Tensor, torch.Tensor, float, float]] = None,
+                  mix: Optional[torch.Tensor] = None, give: Optional[torch.Tensor] = None,
+                  take: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  gather: Optional[torch.Tensor] = None, write: bool = True) -> None:
+    """A pass over the ``count`` streams of the tokens (csrc/hyper_connections.cu; ``streams`` float32 [tokens, count, width]):
+    x_t <- sum_s mix[s, t] x_s + give[t] y, then out = norm(sum_t take[t] x_t) in the type of ``out``. ``single`` (float32
+    [tokens, width]) stands for every old stream. Without ``y`` nothing is mixed in. With ``y2`` and ``y_norms`` = (weight,
+    weight, eps, scale) the output is scale (norm(y) + norm(y2)). ``take`` None: the plain sum; ``norm_weight`` None: no
+    norm. ``gather``: the tokens of the rows, the streams are left alone."""
+    _need(streams, torch.float32, "streams")
+    assert streams.numel() >= rows * count * width and out.is_contiguous() and out.shape[-1] == width
+    for tensor in (single, y2, mix, give, take, norm_weight):
+        if tensor is not None:
+            _need(tensor, torch.float32, "a tensor of hyper_connect")
+    if y is not None:
+        assert y.stride(-1) == 1 and y.shape[-1] == width and mix.numel() == count * count and give.numel() == count
+    assert take is None or take.numel() == count
+    y_w, y2_w, y_eps, y_scale = y_norms if y_norms is not None else (None, None, 0.0, 1.0)
+    assert (y2 is None) == (y_norms is None)
+    _check(library().celeg_hyper_connect(
+        _ptr(single), _ptr(streams), count, int(write and gather is None and y is not None), _ptr(y),
+        dtype_code(y.dtype) if y is not None else FLOAT32, y.stride(0) if y is not None else 0, _ptr(y2),
+        y2.stride(0) if y2 is not None else 0, _ptr(y_w), _ptr(y2_w), y_eps, y_scale, _ptr(mix), _ptr(give), _ptr(take),
+        _ptr(norm_weight), eps, _ptr(out), dtype_code(out.dtype), _ptr(gather), rows, width, _stream()))
+
+
+def normed_pair(a: torch.Tensor, b: torch.Tensor, a_weight: torch.Tensor, b_weight: torch.Tensor, eps: float, scale: float,
+                out: torch.Tensor, rows: int) -> None:
+    """out[:rows] = scale (a / rms(a) * a_weight + b / rms(b) * b_weight), rms(x) = sqrt(mean(x^2) + eps); float32 rows."""
+    for tensor in (a, b, a_weight, b_weight):
+        _need(tensor, torch.float32, "a tensor of normed_pair")
+    assert out.is_contiguous() and a.shape[-1] == b.shape[-1] == out.shape[-1]
+    _check(library().celeg_normed_pair(_ptr(a), _ptr(b), _ptr(a_weight), _ptr(b_weight), eps, scale, _ptr(out),
+                                       dtype_code(out.dtype), rows, out.shape[-1], _stream()))
+
+
+def channel_conv(x: torch.Tensor, kernel: torch.Tensor, bias: Optional[torch.Tensor], carried: Optional[torch.Tensor],
+                 slot_stride: int, token_span: torch.Tensor, span_begin: torch.Tensor, span_slot: torch.Tensor,
+                 out: torch.Tensor, tokens: int, spans: int, act: int = -1, single: bool = False) -> None:
+    """out[t, c] = act(sum_j kernel[c, j] x[t - taps + 1 + j, c] + bias[c]) along every span, with the carried inputs before
+    its start; then the carried inputs [taps - 1, channels] of each request's slot are moved on (csrc/channel_conv.cu).
+    ``x``: float32 columns of wider rows. ``single``: every span is one token."""
+    channels, taps = kernel.shape
+    for tensor in (x, kernel, out):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert kernel.is_contiguous() and x.shape[-1] >= channels and out.shape[-1] >= channels
+    _check(library().celeg_channel_conv(_ptr(x), x.stride(0), _ptr(kernel), _ptr(bias), _ptr(carried), slot_stride,
+                                        _ptr(token_span), _ptr(span_begin), _ptr(span_slot), _ptr(out), out.stride(0), tokens,
+                                        spans, channels, taps, act, int(single), _stream()))
+    global LAUNCHES
+    LAUNCHES += 0 if single or taps == 1 else 1
+
+
+DECAY_MAX_DIM = 256
+
+
+def chunk_tokens() -> int:
+    """Tokens of a chunk of the scans with token-dependent decays."""
+    return int(library().celeg_chunk_tokens())
+
+
+def chunk_plan(span_begin: torch.Tensor, spans: int, max_chunks: int, plan: torch.Tensor) -> None:
+    """The chunks that the step's spans are cut into (plan: int32 [max_chunks + 1 + spans + 1])."""
+    _need(plan, torch.int32, "plan")
+    assert plan.numel() >= max_chunks + spans + 2
+    _check(library().celeg_chunk_plan(_ptr(span_begin), spans, max_chunks, _ptr(plan), _stream()))
+
+
+def channel_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, tau: float,
+                       q_scale: float, q_out: torch.Tensor, k_out: torch.Tensor, total: torch.Tensor, products: torch.Tensor,
+                       states: torch.Tensor, out: torch.Tensor, state: torch.Tensor, slot_stride: int,
+                       span_slot: torch.Tensor, plan: torch.Tensor, max_chunks: int, spans: int, chunks: int, heads: int,
+                       dim: int, vdim: int) -> None:
+    """S <- diag(sigmoid(z + bias)^(1 / tau)) S + k v^T, o = q_scale S^T q along the step's spans (csrc/decayed_scan.cu).
+    ``chunks`` bounds the chunks that the spans make; the scratch holds that many."""
+    for tensor in (q, k, v, z, bias, q_out, k_out, total, products, states, out, state):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert q_out.shape[1] == k_out.shape[1] == heads * dim and out.is_contiguous() and out.shape[1] == heads * vdim
+    assert states.numel() >= chunks * heads * dim * vdim and total.numel() >= chunks * heads * dim
+    assert products.numel() >= chunks * heads * 4096
+    _check(library().celeg_channel_decay_scan(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(z), z.stride(0), _ptr(bias), 1.0 / tau, q_scale,
+        _ptr(q_out), _ptr(k_out), _ptr(total), _ptr(products), _ptr(states), _ptr(out), _ptr(state), slot_stride,
+        _ptr(span_slot), _ptr(plan), max_chunks, spans, chunks, heads, dim, vdim, _stream()))
+    global LAUNCHES
+    LAUNCHES += 3          # the chunks' own products, their states, the carried states, the read-outs
+
+
+def scalar_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Tensor, dt_bias: torch.Tensor,
+                      a_log: torch.Tensor, direct: Optional[torch.Tensor], cum: torch.Tensor, dt: torch.Tensor,
+                      products: torch.Tensor, states: torch.Tensor, out: torch.Tensor, state: torch.Tensor, slot_stride: int,
+                      span_slot: torch.Tensor, plan: torch.Tensor, max_chunks: int, spans: int, chunks: int, heads: int,
+                      groups: int, dim: int, vdim: int) -> None:
+    """S <- exp(-exp(a_log) dt) S + dt k v^T, o = S^T q + direct v with dt = softplus(raw + dt_bias) along the step's spans;
+    heads / groups heads share queries and keys (csrc/decayed_scan.cu)."""
+    for tensor in (q, k, v, raw, dt_bias, a_log, cum, dt, products, states, out, state):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert out.is_contiguous() and out.shape[1] == heads * vdim and states.numel() >= chunks * heads * dim * vdim
+    assert products.numel() >= chunks * groups * 4096
+    _check(library().celeg_scalar_decay_scan(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(raw), raw.stride(0), _ptr(dt_bias), _ptr(a_log),
+        _ptr(direct), _ptr(cum), _ptr(dt), _ptr(products), _ptr(states), _ptr(out), _ptr(state), slot_stride, _ptr(span_slot),
+        _ptr(plan), max_chunks, spans, chunks, heads, groups, dim, vdim, _stream()))
+    global LAUNCHES
+    LAUNCHES += 4          # the decays, the products, then as above
+
+
+def channel_decay_decode(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_scale: float, low: torch.Tensor,
+                         up: torch.Tensor, bias: torch.Tensor, tau: float, norm_weight: torch.Tensor, eps: float,
+                         gate: torch.Tensor, state: torch.Tensor, slot_stride: int, span_slot: torch.Tensor, tokens: int,
+                         heads: int, dim: int, vdim: int, out: torch.Tensor) -> None:
+    """A decoding step of the channel form in one launch: the decay's second product (``low`` float32 rows, ``up`` [heads *
+    dim, rank] in the type of ``out``), state update, read-out, the heads' norm (``norm_weight`` [vdim]) and SiLU gate."""
+    for tensor in (q, k, v, low, bias, norm_weight, gate, state):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert up.dtype == out.dtype and up.is_contiguous() and up.shape[0] == heads * dim
+    assert out.is_contiguous() and out.shape[1] == heads * vdim
+    _check(library().celeg_channel_decay_decode(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), q_scale, _ptr(low), low.stride(0), _ptr(up),
+        up.shape[1], _ptr(bias), 1.0 / tau, _ptr(norm_weight), eps, _ptr(gate), gate.stride(0), _ptr(state), slot_stride,
+        _ptr(span_slot), tokens, heads, dim, vdim, _ptr(out), dtype_code(out.dtype), _stream()))
+
+
+def scalar_decay_decode(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Tensor, dt_bias: torch.Tensor,
+                        a_log: torch.Tensor, direct: Optional[torch.Tensor], state: torch.Tensor, slot_stride: int,
+                        span_slot: torch.Tensor, tokens: int, heads: int, groups: int, dim: int, vdim: int,
+                        out: torch.Tensor) -> None:
+    """A decoding step of the scalar form: state update and read-out (float32, the values' direct share added)."""
+    for tensor in (q, k, v, raw, dt_bias, a_log, state, out):
+        assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
+    assert out.is_contiguous() and out.shape[1] == heads * vdim
+    _check(library().celeg_scalar_decay_decode(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(raw), raw.stride(0), _ptr(dt_bias), _ptr(a_log),
+        _ptr(direct), _ptr(state), slot_stride, _ptr(span_slot), tokens, heads, groups, dim, vdim, _ptr(out), _stream()))

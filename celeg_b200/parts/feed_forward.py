@@ -21,22 +21,32 @@ ACTIVATIONS = {"gelu": kernels.ACT_GELU_ERF, "gelu_tanh": kernels.ACT_GELU_TANH,
 GATE_FORMS = {"clamped_silu": kernels.GATE_CLAMPED_SILU}
 
 
+def gate_constants(name: str, params: Mapping):
+    """(limit, slope, shift) of the clamped form, zeros for every other function of a gate."""
+    if name != "clamped_silu":
+        return kernels.NO_GATE_CONSTANTS
+    return float(params["gate_limit"]), float(params.get("gate_slope", 1.0)), float(params.get("up_shift", 0.0))
+
+
 @register_part("feed_forward", "swiglu")
 class SwiGluFeedForward:
     """down(silu(gate(x)) * up(x)); gate and up are one fused projection [2I, H] (gate rows
     first), as celeg concatenates w1 and w3 (src/backend/cpu/weights_loader.cpp:93-99;
     src/backend/cuda/packed/operators.cu:531-596). ``activation`` names another function of the gate (a gated
-    linear unit with ReLU, a GELU, ...): in the weight-streaming product's epilogue for steps of few rows, else as the
-    product and an element-wise kernel."""
+    linear unit with ReLU, a GELU, ...), "clamped_silu" the form g sigmoid(``gate_slope`` g) (u + ``up_shift``) of a gate
+    cut off at ``gate_limit`` and an up value cut off at both signs of it: in the weight-streaming product's epilogue for
+    steps of few rows, in the tcgen05 product's for very many, else as the product and an element-wise kernel."""
 
     def __init__(self, params: Mapping, weights: Mapping[str, torch.Tensor], parts: Mapping, rt: Runtime):
         self.rt = rt
         self.hidden = int(params["hidden_size"])
         self.inner = int(params["intermediate_size"])
         name = params.get("activation", "silu")
-        if name not in ACTIVATIONS:
-            raise ValueError(f"gated feed-forward: unknown activation {name!r}; known: {', '.join(ACTIVATIONS)}")
-        self.activation = ACTIVATIONS[name]
+        known = dict(ACTIVATIONS, **GATE_FORMS)
+        if name not in known:
+            raise ValueError(f"gated feed-forward: unknown activation {name!r}; known: {', '.join(known)}")
+        self.activation = known[name]
+        self.gate_constants = gate_constants(name, params)
         self.w_gate_up = rt.matrix(torch.cat([weights["gate"], weights["up"]], dim=0))
         self.w_down = rt.matrix(weights["down"])
         self.gate_up = rt.scratch("swiglu.gate_up", 2 * self.inner)
@@ -49,7 +59,8 @@ class SwiGluFeedForward:
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
         rt, t = self.rt, step.tokens
-        rt.linear_swiglu(x, self.w_gate_up, self.gate_up, self.activated, t, self.inner, self.activation)
+        rt.linear_swiglu(x, self.w_gate_up, self.gate_up, self.activated, t, self.inner, self.activation,
+                         self.gate_constants)
         rt.linear(self.activated, self.w_down, out, t)
 
 
@@ -116,10 +127,7 @@ class MoeFeedForward:
         if name not in known:
             raise ValueError(f"moe: unknown activation {name!r}; known: {', '.join(known)}")
         self.activation = known[name]
-        self.gate_constants = kernels.NO_GATE_CONSTANTS
-        if name == "clamped_silu":
-            self.gate_constants = (float(params["gate_limit"]), float(params.get("gate_slope", 1.0)),
-                                   float(params.get("up_shift", 0.0)))
+        self.gate_constants = gate_constants(name, params)
         scores = params.get("scores", "softmax")
         if scores not in ("softmax", "sigmoid"):
             raise ValueError(f"moe: unknown scores {scores!r}; known: softmax, sigmoid")

@@ -108,7 +108,7 @@ class PagedAttentionKernels:
     """The choice among the attention kernels for a step's queries over a paged cache, shared by the mixers that
     attend over one. A mixer that inherits it has ``rt``, ``heads``, ``kv_heads``, ``head_dim``, ``window``, ``scale``,
     ``sinks`` (or None), ``distance_bias`` (absent, None, or a float32 table [heads, n + 1] of score biases by distance
-    back to the key), ``binding``, the queries in ``qkv`` (head h of a row at h * head_dim, rows ``qkv_width``
+    back to the key), ``softcap`` (absent, None, or what scaled scores are capped at, softly), ``binding``, the queries in ``qkv`` (head h of a row at h * head_dim, rows ``qkv_width``
     apart), the output buffer ``attended`` [tokens, heads * head_dim] and ``_resident_blocks = None``.
     ``_value_cache()`` names the tensor the values are read from: the binding's own, or the keys themselves for a
     mixer whose values are a leading part of what it caches as keys."""
@@ -175,7 +175,8 @@ class PagedAttentionKernels:
                                  step.token_span, table, count, self.heads, self.kv_heads,
                                  self.head_dim, b.page_tokens, self._mask(), self.scale, chunk, max_splits,
                                  partial_o, partial_ml, counters, step.error_flag, sinks=self.sinks,
-                                 distance_bias=getattr(self, "distance_bias", None))
+                                 distance_bias=getattr(self, "distance_bias", None),
+                                 softcap=getattr(self, "softcap", None))
 
     def _attend_portions(self, step: StepContext, table: torch.Tensor, skip: int) -> None:
         """The spans from ``skip`` on (the spans before it have one token each, so span ``skip`` begins at token
@@ -196,13 +197,15 @@ class PagedAttentionKernels:
                                               span_begin, span_table, step.tokens, spans, tiles, self.heads,
                                               self.kv_heads, self.head_dim, b.page_tokens, self._mask(), self.scale,
                                               step.error_flag, sinks=self.sinks,
-                                              distance_bias=getattr(self, "distance_bias", None))
+                                              distance_bias=getattr(self, "distance_bias", None),
+                                              softcap=getattr(self, "softcap", None))
             return
         if kernels.attention_prefill_supported(self.heads, self.kv_heads, self.head_dim, rt.act_dtype):
             kernels.attention_prefill(self.qkv, self.qkv_width, self.attended, b.k, values, step.positions,
                                       span_begin, span_table, step.tokens, spans, self.heads, self.kv_heads,
                                       self.head_dim, b.page_tokens, self._mask(), self.scale, step.error_flag,
-                                      sinks=self.sinks, distance_bias=getattr(self, "distance_bias", None))
+                                      sinks=self.sinks, distance_bias=getattr(self, "distance_bias", None),
+                                      softcap=getattr(self, "softcap", None))
             return
         self._attend_general(step, table, skip)
 
@@ -218,7 +221,8 @@ class PagedAttentionKernels:
                                   step.positions[skip:], step.token_span[skip:], table, step.tokens - skip,
                                   self.heads, self.kv_heads, self.head_dim, b.page_tokens, self.window, self.scale,
                                   step.error_flag, sinks=self.sinks, value_dim=getattr(self, "value_dim", None),
-                                  chunk=getattr(self, "chunk", None), distance_bias=getattr(self, "distance_bias", None))
+                                  chunk=getattr(self, "chunk", None), distance_bias=getattr(self, "distance_bias", None),
+                                  softcap=getattr(self, "softcap", None))
 
 
 @register_part("mixer", "attention")
@@ -368,12 +372,32 @@ def distance_bias_table(table: torch.Tensor, far: int) -> torch.Tensor:
     return table.to(torch.float32)[rows].t().contiguous()
 
 
+class CarriedInputs:
+    """The state of a mixer's short convolutions where the mixer itself holds keys and values: the last taps - 1 inputs of
+    ``channels`` channels, a cache part of its own under the mixer's name (see ``children`` of a part)."""
+
+    def __init__(self, channels: int, taps: int):
+        self.channels, self.taps = channels, taps
+        self.state: Optional[torch.Tensor] = None
+        self.slot_stride = 0
+
+    def cache_need(self):
+        return StateNeed(elements=(self.taps - 1) * self.channels) if self.taps > 1 else None
+
+    def bind_cache(self, binding: StateBinding) -> None:
+        self.state, self.slot_stride = binding.state, binding.slot_stride
+
+
 @register_part("mixer", "prepared_attention")
 class PreparedAttentionMixer(PagedAttentionKernels):
     """Causal grouped-query softmax attention whose q, k and v leave one fused projection as float32 sums and are
     made ready for the paged attention kernels by one launch. Everything but the four matrices is optional:
 
     * biases on the projections (tensors ``q_bias``, ``k_bias``, ``v_bias``, ``out_bias``);
+    * ``taps``: a causal convolution over time on every channel of q, k and v as projected (tensors ``q_conv``, ``k_conv``,
+      ``v_conv`` [channels, taps], the last tap for the token itself), before everything below; the last taps - 1 projected
+      rows of a request are its state;
+    * ``softcap`` = c: scaled scores s become c tanh(s / c);
     * ``whole_qk_norm``: one RMS norm over the whole q projection and one over the whole k projection (tensors
       ``q_norm``, ``k_norm`` as wide as the projections, ``eps``); or ``head_qk_norm``: one a head, with weights as wide
       as a head that all heads share;
@@ -456,6 +480,22 @@ class PreparedAttentionMixer(PagedAttentionKernels):
             if self.gate_per_head and self.heads % 8:       # (zero rows: the projection's rows stay 16-byte aligned)
                 stacked.append(torch.zeros((-self.heads % 8, self.hidden), dtype=gate_rows.dtype))
         self.w_qkv = rt.matrix(torch.cat(stacked, dim=0))
+        cap = params.get("softcap")
+        self.softcap = float(cap) if cap else None
+        if self.softcap is not None and self.softcap < 0:
+            raise ValueError(f"attention: scores capped at {self.softcap}")
+        taps = params.get("taps")
+        self.conv = self.conv_kernel = self.convolved = None
+        if taps:
+            if self.reads_only or {"q_bias", "k_bias", "v_bias"} & set(weights):
+                raise ValueError("attention: short convolutions need keys and values of the mixer's own and no biases before them")
+            if not 1 <= int(taps) <= 16:
+                raise ValueError(f"attention: {taps} taps (1 to 16)")
+            self.conv_kernel = rt.vector(torch.cat([weights[name + "_conv"].reshape(width, int(taps)) for name, width in
+                                                    (("q", q_width), ("k", k_width), ("v", v_width))], dim=0))
+            self.conv = CarriedInputs(q_width + k_width + v_width, int(taps))
+            self.convolved = rt.scratch("prepared_attention.conv", self.conv.channels, torch.float32)
+            self.children = {"conv": self.conv}
         biases = [weights.get("q_bias"), weights.get("k_bias"), weights.get("v_bias")]
         if any(b is not None for b in biases):
             widths = (q_width, k_width, v_width)
@@ -547,9 +587,15 @@ class PreparedAttentionMixer(PagedAttentionKernels):
         rt, b, t = self.rt, self.binding, step.tokens
         rt.linear(x, self.w_qkv, self.projected, t)
         table = step.block_tables[b.group]
+        rows = self.projected
+        if self.conv is not None:
+            kernels.channel_conv(rows, self.conv_kernel, None, self.conv.state, self.conv.slot_stride, step.token_span,
+                                 step.span_begin, step.span_slot, self.convolved, t, step.spans,
+                                 single=step.max_span == 1 and step.spans == t)
+            rows = self.convolved
         if self.prepares:
             k_pages, v_pages, kv_heads = (None, None, 0) if self.reads_only else (b.k, b.v, self.kv_heads)
-            kernels.qkv_prepare(self.projected, self.bias, self.qkv, step.positions, step.token_span, table, k_pages, v_pages,
+            kernels.qkv_prepare(rows, self.bias, self.qkv, step.positions, step.token_span, table, k_pages, v_pages,
                                 t, self.heads, kv_heads, self.dim, self.vdim, self.head_dim, self.value_dim,
                                 b.page_tokens, step.error_flag, q_norm=self.q_norm, k_norm=self.k_norm,
                                 norm_eps=self.eps, norm_per_head=self.head_qk_norm,
@@ -558,7 +604,7 @@ class PreparedAttentionMixer(PagedAttentionKernels):
                                 temperature=self.temperature, blend=self.blend, lam=self.lam,
                                 first_values=self.first_values)
         else:
-            kernels.bias_store_kv(self.projected, self.bias, self.qkv, step.positions, step.token_span, table, b.k, b.v,
+            kernels.bias_store_kv(rows, self.bias, self.qkv, step.positions, step.token_span, table, b.k, b.v,
                                   t, self.heads, self.kv_heads, self.dim, self.vdim, self.head_dim, self.value_dim,
                                   b.page_tokens, step.error_flag)
         self.attend(step, table)
@@ -592,7 +638,8 @@ class ChunkedAttentionMixer(PreparedAttentionMixer):
 @register_part("mixer", "side_by_side")
 class SideBySideMixer:
     """Two mixers (nested parts ``left`` and ``right``) that read the same rows; the result is
-    left_scale * left + right_scale * right. Each child leaves its result as float32 rows (its last product's sums);
+    left_scale * left + right_scale * right, with the tensors ``left_norm`` and ``right_norm`` (the model's width, ``eps``)
+    of both outputs RMS-normed first. Each child leaves its result as float32 rows (its last product's sums);
     one launch scales, adds (a child's output bias too, if it hands one over) and rounds once. A child that holds
     a cache gets its own: the children are named to the model under ``children``."""
 
@@ -607,6 +654,10 @@ class SideBySideMixer:
         self.children = {"left": self.left, "right": self.right}
         self.left_out = rt.scratch("side_by_side.left", self.hidden, torch.float32)
         self.right_out = rt.scratch("side_by_side.right", self.hidden, torch.float32)
+        self.norms = None                                  # (weight, weight, eps), the scales in the weights
+        if "left_norm" in weights or "right_norm" in weights:
+            self.norms = (rt.vector(weights["left_norm"]).mul_(self.left_scale),
+                          rt.vector(weights["right_norm"]).mul_(self.right_scale), float(params["eps"]))
 
     @staticmethod
     def _run(child, x, out, step):
@@ -616,9 +667,42 @@ class SideBySideMixer:
         child.forward(x, out, step)
         return None
 
-    def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
+    def _run_both(self, x, step: StepContext):
+        """Both children's rows; returns their output biases (or None)."""
+        rt = self.rt
+        if not (rt.side_by_side_branches and rt.small_batch(step.tokens)):
+            return self._run(self.left, x, self.left_out, step), self._run(self.right, x, self.right_out, step)
+        # few rows: two chains of short kernels that share nothing but their input; the second goes to a second stream
+        # (two branches of the step's graph when it is captured) and is joined before anything reads the results
+        main, side = torch.cuda.current_stream(rt.device), rt.side_stream()
+        fork = torch.cuda.Event()
+        fork.record(main)
+        side.wait_event(fork)
+        with torch.cuda.stream(side):
+            right_bias = self._run(self.right, x, self.right_out, step)
+            join = torch.cuda.Event()
+            join.record(side)
         left_bias = self._run(self.left, x, self.left_out, step)
-        right_bias = self._run(self.right, x, self.right_out, step)
+        main.wait_event(join)
+        return left_bias, right_bias
+
+    def forward_normed_pair(self, x: torch.Tensor, step: StepContext):
+        """forward() without its last pass, for a caller that forms it in a pass of its own: (left rows, right rows, (weight,
+        weight, eps)), the result being the sum of the two normed rows. None: the outputs are not normed."""
+        if self.norms is None:
+            return None
+        left_bias, right_bias = self._run_both(x, step)
+        for bias, rows in ((left_bias, self.left_out), (right_bias, self.right_out)):
+            if bias is not None:
+                kernels.scaled_sum(rows, None, bias, 1.0, 0.0, rows, step.tokens)
+        return self.left_out, self.right_out, self.norms
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
+        if self.norms is not None:
+            left, right, (left_weight, right_weight, eps) = self.forward_normed_pair(x, step)
+            kernels.normed_pair(left, right, left_weight, right_weight, eps, 1.0, out, step.tokens)
+            return
+        left_bias, right_bias = self._run_both(x, step)
         if right_bias is not None and left_bias is None:
             kernels.scaled_sum(self.right_out, self.left_out, right_bias, self.right_scale, self.left_scale, out, step.tokens)
             return

@@ -1,7 +1,7 @@
 """Registries of part kinds. A model description names parts by ``kind``; the class behind a
 kind is looked up here when the model is built, so a new mixer, feed-forward, norm, position
-encoding, block arrangement, end of the model (what makes rows of token ids, what makes logits of rows) or
-part that rewrites the stream between two blocks is added by registering a class, with no change to the engine.
+encoding, block arrangement, end of the model (what makes rows of token ids, what makes logits of rows),
+part that rewrites the stream between two blocks or connection of a sublayer with several streams is added by registering a class, with no change to the engine.
 
 celeg dispatches over closed variants (``std::visit`` in src/backend/cuda/packed/layer_executor.cu:131-191);
 the open registry is this engine's own choice.
@@ -10,7 +10,7 @@ from __future__ import annotations
 
 from typing import Callable, Dict
 
-CATEGORIES = ("norm", "mixer", "feed_forward", "position", "arrangement", "input", "output", "stream")
+CATEGORIES = ("norm", "mixer", "feed_forward", "position", "arrangement", "input", "output", "stream", "connection")
 _REGISTRY: Dict[str, Dict[str, Callable]] = {category: {} for category in CATEGORIES}
 
 

@@ -50,6 +50,8 @@ class ResidualStream:
         self.rows = rt.scratch("stream.rows", hidden) if rt.act_dtype != torch.float32 else self.residual
         self.rows_current = False
         self.wants_rows = False
+        # several streams in place of one (parts/hyper_connections.py): while they are open the stream is theirs
+        self.copies = None
         self.pieces = (hidden + 15) // 16
         if rt.act_dtype == torch.bfloat16:
             self.xw = rt.scratch("stream.split_norm", hidden, torch.bfloat16)
@@ -64,6 +66,8 @@ class ResidualStream:
         self.ready = None
         self.rows_current = False
         self.rt.sink = None
+        if self.copies is not None:
+            self.copies.close()
 
     def as_rows(self, rows: int) -> torch.Tensor:
         """The stream's first ``rows`` rows in the activation type, with everything owed to it added: what a sublayer
@@ -107,6 +111,9 @@ class ResidualStream:
         """out = norm(stream + pending) for the first ``rows`` rows (or the gathered ones). Without
         ``gather`` what was pending is added for good. Returns ``out``, or the split norm that the
         last product prepared for exactly this norm."""
+        if self.copies is not None and self.copies.open:
+            self.copies.total(out, rows, norm=norm, gather=gather)
+            return out
         if self.prepared is not None:
             prepared_norm, split = self.prepared
             self.prepared = None
@@ -146,6 +153,8 @@ class ResidualStream:
 
     def settle(self, rows: int) -> None:
         """Add what is owed to the stream now (for a reader that wants the stream itself)."""
+        if self.copies is not None and self.copies.open:
+            raise RuntimeError("the stream is several streams: a part that wants it as one row a token cannot run here")
         if self.pending is not None or self.pending_b is not None:
             self.rows_current = False
             kernels.add_to_residual(self.residual, self.pending, self.pending_b, rows)
@@ -337,9 +346,10 @@ class Runtime:
                 torch.mm(x[:padded], weight.t(), out=out[:padded])
 
     def linear_swiglu(self, x: torch.Tensor, gate_up_weight: torch.Tensor, scratch: torch.Tensor,
-                      out: torch.Tensor, rows: int, inner: int, kind: int = kernels.ACT_SILU) -> None:
+                      out: torch.Tensor, rows: int, inner: int, kind: int = kernels.ACT_SILU,
+                      constants: Tuple[float, float, float] = kernels.NO_GATE_CONSTANTS) -> None:
         """out[:rows] = act(x gate^T) * (x up^T) with gate_up_weight = [gate rows; up rows], act = SiLU or the
-        ``kind`` given (a code of kernels.ACT_*). Few bfloat16 rows: one weight-streaming kernel; very many
+        ``kind`` given (a code of kernels.ACT_*, or kernels.GATE_CLAMPED_SILU with its ``constants``). Few bfloat16 rows: one weight-streaming kernel; very many
         bfloat16 rows: one tcgen05 kernel (the gate's function in its epilogue); otherwise the product into ``scratch`` and the element-wise
         kernel."""
         if rows == 0:
@@ -347,7 +357,8 @@ class Runtime:
         operand = x.xw if isinstance(x, kernels.SplitNorm) else x
         if self.act_dtype == torch.bfloat16 and kernels.gemv_supported(rows, operand, gate_up_weight):
             kernels.gemv_bf16(x, gate_up_weight, out, rows, kernels.GEMV_SWIGLU, ahead=self._ahead(gate_up_weight),
-                              taps=0 if kind == kernels.ACT_SILU else 1 + kind)
+                              taps=0 if kind == kernels.ACT_SILU else 1 + kind,
+                              gate_constants=constants if kind == kernels.GATE_CLAMPED_SILU else None)
             return
         if (self.act_dtype == torch.bfloat16 and kernels.gemm_tcgen05_supported(x, gate_up_weight)
                 and (self.tensor_core_products == "all"
@@ -355,11 +366,11 @@ class Runtime:
                          and gate_up_weight.shape[1] >= self.tensor_core_min_width))):
             kernels.gemm_tcgen05(x, gate_up_weight, out, rows,
                                  kernels.TC_SWIGLU if kind == kernels.ACT_SILU else kernels.TC_GATED + kind,
-                                 self.error_flag, self.tensor_core_variant)
+                                 self.error_flag, self.tensor_core_variant, constants)
             return
         self.linear(x, gate_up_weight, scratch, rows)
         if kind != kernels.ACT_SILU:
-            kernels.glu(scratch, out, rows, inner, kind)
+            kernels.glu(scratch, out, rows, inner, kind, constants)
         else:
             kernels.swiglu(scratch, out, rows, inner)
 
