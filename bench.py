@@ -8,7 +8,7 @@ batch 1 and 64. Prints ONE JSON line.
                   [--prefill-tokens T] [--chunk C] [--kernel-times] [--no-cuda-graph]      one phase, a short record
   python bench.py --workload lfm2-700m|lfm2-350m [--requests N] [--new-tokens N] [--max-batched-tokens N]
                   [--prefill-chunk N] [--kernel-times]       a scheduler workload through Engine.submit/step/poll
-  python bench.py --design ramosun|kedesun|naselorn|liverax|kodupel [--design-size w1024|w2048] [--kernel-times]
+  python bench.py --design ramosun|kedesun|naselorn|liverax|kodupel|fovezen [--design-size w1024|w2048] [--kernel-times]
                   the Ramosun design beside the closest LFM2 model at equal size: prefill of 2,048 tokens, decode at batch 8
 
 A "step" is one decode step of the whole batch. ``value`` is timed on the device (CUDA events
@@ -199,7 +199,9 @@ class KernelTimer:
              "expert_product", "expert_product_tcgen05", "expert_rows", "moe_combine", "retention_segmented",
              "retention_decode_raw", "activation_columns", "bias_store_kv", "scaled_sum", "glu", "lru_prepare",
              "block_diagonal_product", "lru_scan", "lru_decode", "add_layernorm", "qkv_prepare", "rmsnorm_strided",
-             "sigmoid_gate", "output_norm", "activation_cast", "general_delta_scan", "general_delta_decode")
+             "sigmoid_gate", "output_norm", "activation_cast", "general_delta_scan", "general_delta_decode",
+             "hyper_connect", "normed_pair", "channel_conv", "chunk_plan", "channel_decay_scan", "scalar_decay_scan",
+             "channel_decay_decode", "scalar_decay_decode")
 
     def __init__(self):
         self.pairs = []
@@ -562,6 +564,29 @@ def kodupel_config(width: int, vocab: int) -> dict:
             "layers": layers, "max_context": 8192}
 
 
+def fovezen_config(width: int, vocab: int) -> dict:
+    """Six layers over four streams, the second and third twice (eight layers run): Mamba-2, side by side, rotary attention,
+    Mamba-2, side by side, Mamba-2. The Mamba-2 mixer has twice as many channels as the model is wide in heads of 64 with
+    states of 128, eight groups and norm groups; the left half of the side-by-side mixer has query heads of 64 on a quarter
+    as many key heads under a window of 1,024 positions with capped scores, the right half the lightning mixer's sizes
+    (heads of 64 keys and 128 values) with a decay of rank width / 32; the rotary attention has heads of 128; a clamped
+    gated feed-forward of 8/3 width."""
+    heads = width // 64
+    ff = {"kind": "dense", "ff": (8 * width // 3 + 127) // 128 * 128, "limit": 7.0}
+    mamba = {"type": "mamba2", "mlp": ff, "mixer": {"heads": 2 * heads, "vdim": 64, "state": 128, "groups": 8, "conv": 4,
+                                                    "norm_groups": 8}}
+    parallel = {"type": "parallel", "mlp": ff, "mixer": {
+        "left": {"heads": heads, "kv_heads": heads // 4, "dim": 64, "vdim": 64, "scale": 0.125, "conv": 4, "softcap": 30.0,
+                 "mask": {"size": 1024}},
+        "right": {"heads": heads // 2, "dim": 64, "vdim": 128, "tau": 16.0, "decay_rank": width // 32}}}
+    attention = {"type": "attention", "mlp": ff, "mixer": {
+        "heads": heads // 2, "kv_heads": max(heads // 8, 1), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+        "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}}
+    return {"architecture": "Fovezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": 4, "logit_scale": 0.5,
+            "layers": [mamba, parallel, attention, mamba, parallel, mamba], "loop": {"start": 1, "stop": 3, "times": 2},
+            "max_context": 8192}
+
+
 def lfm2_attention_only(width: int, vocab: int) -> dict:
     """The LFM2 relative with attention in all eight blocks: the existing model closest to a design whose mixers are all
     softmax attention (pre-norm blocks, grouped queries, rotation of halves, a gated feed-forward)."""
@@ -603,6 +628,9 @@ def run_design(args) -> dict:
                       ("kedesun", kedesun_config(width, vocab)))
         elif args.design == "kodupel":   # beside Naselorn (gated experts) and Ramosun (a delta rule, per-head state)
             models = (("kodupel", kodupel_config(width, vocab)), ("naselorn", naselorn_config(width, vocab)),
+                      ("ramosun", ramosun_config(width, vocab)))
+        elif args.design == "fovezen":   # beside Naselorn (side-by-side mixers, matrix states) and Ramosun (convolutions, a loop)
+            models = (("fovezen", fovezen_config(width, vocab)), ("naselorn", naselorn_config(width, vocab)),
                       ("ramosun", ramosun_config(width, vocab)))
         else:
             models = (("ramosun", ramosun_config(width, vocab)), ("lfm2", lfm2_relative(width, vocab)))
@@ -885,7 +913,7 @@ def main() -> int:
     parser.add_argument("--new-tokens", type=int, default=0, help="--workload: tokens to generate per request")
     parser.add_argument("--max-batched-tokens", type=int, default=0, help="--workload: token budget of a step")
     parser.add_argument("--prefill-chunk", type=int, default=0, help="--workload: longest prompt portion")
-    parser.add_argument("--design", default=None, choices=["ramosun", "kedesun", "naselorn", "liverax", "kodupel"],
+    parser.add_argument("--design", default=None, choices=["ramosun", "kedesun", "naselorn", "liverax", "kodupel", "fovezen"],
                         help="prefill and decode of that design beside the closest LFM2 model at equal size")
     parser.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="--design: one size only")
     parser.add_argument("--no-warmup-run", action="store_true",

@@ -9,7 +9,7 @@
 
 namespace celeg_b200 {
 
-constexpr int kConvTile = 8;          // tokens a thread walks
+constexpr int kConvTile = 4;          // tokens a thread walks (portions; a decoded token has a thread of its own)
 
 struct ChannelConvArgs {
     const float* in; int in_stride;
@@ -43,12 +43,12 @@ template <int V> __device__ __forceinline__ void conv_store(float* p, const Conv
 }
 
 // V neighbouring channels a thread, TAPS taps (a template for up to four; 16: any number up to that)
-template <int V, int TAPS>
+template <int V, int TAPS, int TILE>
 __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvArgs a) {
     const int taps = TAPS <= 4 ? TAPS : a.taps;
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
-    const int t0 = blockIdx.y * (TAPS <= 4 ? kConvTile : 1);
-    const int t1 = min(t0 + (TAPS <= 4 ? kConvTile : 1), a.tokens);
+    const int t0 = blockIdx.y * (TAPS <= 4 ? TILE : 1);
+    const int t1 = min(t0 + (TAPS <= 4 ? TILE : 1), a.tokens);
     chain_release();
     chain_wait();
     if (c >= a.channels) return;
@@ -56,8 +56,13 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvArgs
     if constexpr (TAPS <= 4) {
 #pragma unroll
         for (int i = 0; i < V; ++i)
+            if (TAPS == 4) {
+                const float4 x = __ldg(reinterpret_cast<const float4*>(a.w) + c + i);
+                w[0][i] = x.x; w[1 % TAPS][i] = x.y; w[2 % TAPS][i] = x.z; w[3 % TAPS][i] = x.w;
+            } else {
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) w[j][i] = __ldg(a.w + (size_t)(c + i) * TAPS + j);
+                for (int j = 0; j < TAPS; ++j) w[j][i] = __ldg(a.w + (size_t)(c + i) * TAPS + j);
+            }
     }
     ConvPack<V> bias;
 #pragma unroll
@@ -72,16 +77,18 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvArgs
     if constexpr (TAPS <= 4) {
         constexpr int kKeep = TAPS > 1 ? TAPS - 1 : 1;
         ConvPack<V> history[kKeep];
-        ConvPack<V> ahead[kConvTile];
+        ConvPack<V> ahead[TILE];
 #pragma unroll
-        for (int i = 0; i < kConvTile; ++i)
+        for (int i = 0; i < TILE; ++i)
             if (t0 + i < t1) ahead[i] = conv_load<V>(a.in + (size_t)(t0 + i) * a.in_stride + c);
         int span = -1;
+        const int last_span = TAPS > 1 ? a.token_span[t1 - 1] : 0;
 #pragma unroll
-        for (int i = 0; i < kConvTile; ++i) {
+        for (int i = 0; i < TILE; ++i) {
             const int t = t0 + i;
             if (t >= t1) continue;
-            if (TAPS > 1 && a.token_span[t] != span) {         // the tile's first token, or a span that begins here
+            // the tile's first token, or a span that begins here (only where the tile's last token is of a later span)
+            if (TAPS > 1 && (i == 0 || (span != last_span && a.token_span[t] != span))) {
                 span = a.token_span[t];
                 const int begin = a.span_begin[span];
                 const float* carried = a.carried + (long long)a.span_slot[span] * a.slot_stride;
@@ -157,17 +164,17 @@ __global__ void channel_conv_carry_kernel(const ChannelConvArgs a, int spans) {
         if (r < a.taps - 1) mine[(size_t)r * a.channels + c] = keep[r];
 }
 
-template <int V>
+template <int V, int TILE>
 static void launch_conv(const ChannelConvArgs& a, cudaStream_t stream) {
-    const int tile = a.taps <= 4 ? kConvTile : 1;
+    const int tile = a.taps <= 4 ? TILE : 1;
     const int units = a.channels / V;
     dim3 grid((units + 127) / 128, (a.tokens + tile - 1) / tile);
     switch (a.taps) {
-        case 1: launch_chained(channel_conv_kernel<V, 1>, grid, 128, 0, stream, a); break;
-        case 2: launch_chained(channel_conv_kernel<V, 2>, grid, 128, 0, stream, a); break;
-        case 3: launch_chained(channel_conv_kernel<V, 3>, grid, 128, 0, stream, a); break;
-        case 4: launch_chained(channel_conv_kernel<V, 4>, grid, 128, 0, stream, a); break;
-        default: launch_chained(channel_conv_kernel<V, 16>, grid, 128, 0, stream, a);
+        case 1: launch_chained(channel_conv_kernel<V, 1, TILE>, grid, 128, 0, stream, a); break;
+        case 2: launch_chained(channel_conv_kernel<V, 2, TILE>, grid, 128, 0, stream, a); break;
+        case 3: launch_chained(channel_conv_kernel<V, 3, TILE>, grid, 128, 0, stream, a); break;
+        case 4: launch_chained(channel_conv_kernel<V, 4, TILE>, grid, 128, 0, stream, a); break;
+        default: launch_chained(channel_conv_kernel<V, 16, TILE>, grid, 128, 0, stream, a);
     }
 }
 
@@ -182,7 +189,7 @@ CELEG_API int celeg_channel_conv(const float* in, int in_stride, const float* w,
                                  float* out, int out_stride, int tokens, int spans, int channels, int taps, int act,
                                  int single, cudaStream_t stream) {
     CELEG_REQUIRE(tokens >= 0 && spans >= 0 && channels > 0 && taps >= 1 && taps <= 16 && in_stride >= channels &&
-                  out_stride >= channels && act >= -1 && act <= kTanh && (taps == 1 || carried),
+                  out_stride >= channels && act >= -1 && act <= kTanh && (taps == 1 || carried) && ((size_t)w & 15) == 0,
                   "channel_conv: invalid sizes tokens=%d channels=%d taps=%d strides %d / %d act=%d", tokens, channels, taps,
                   in_stride, out_stride, act);
     CELEG_REQUIRE(tokens <= 65535, "channel_conv: %d tokens exceed one launch", tokens);
@@ -190,8 +197,8 @@ CELEG_API int celeg_channel_conv(const float* in, int in_stride, const float* w,
     const ChannelConvArgs a = {in, in_stride, w, bias, carried, slot_stride, token_span, span_begin, span_slot, out, out_stride,
                                tokens, channels, taps, act, single};
     if (((channels | in_stride | out_stride) & 3) == 0 && (slot_stride & 3) == 0 &&
-        (((size_t)in | (size_t)out | (size_t)carried) & 15) == 0) launch_conv<4>(a, stream);
-    else launch_conv<1>(a, stream);
+        (((size_t)in | (size_t)out | (size_t)carried) & 15) == 0) single ? launch_conv<4, 1>(a, stream) : launch_conv<4, kConvTile>(a, stream);
+    else single ? launch_conv<1, 1>(a, stream) : launch_conv<1, kConvTile>(a, stream);
     const int status = check_launch("channel_conv");
     if (status != 0 || single || taps == 1) return status;
     const long long units = (long long)spans * channels;

@@ -16,10 +16,11 @@
 // so all chunks are worked on side by side but for one element-wise walk over their states:
 //
 //   prepare   what the chunk's tokens do to one another, and the vectors q P(1..), k P(..n). Scalar: the running sums of
-//             the decays' logarithms; products of decays are exponentials of differences of those. Channel: a chunk's
-//             products in shared memory. A decay may be as good as zero, so nothing is divided by a product: the 64 tokens
-//             are four blocks of 16, the sums within a block carry k_j from token to token, and between blocks both sides
-//             are taken to the border of the later block, where every factor is at most one.
+//             the decays' logarithms; products of decays are exponentials of differences of those. Channel: the 64 tokens
+//             are eight blocks of eight, and within a block queries and keys are taken to its middle, q_i P(5..i) or
+//             q_i / P(i+1..4), k_j P(j+1..4) or k_j / P(5..j): at most four decays are divided by, and as a decay below
+//             1e-8 counts as 1e-8 (the old state's share is then below float32's rounding) that stays within range. The
+//             sums are one small product; between two blocks it has one more factor a channel, a product of decays.
 //   states    sum_j (k_j P(j+1..n)) v_j^T of every chunk, a 64 x 64 tile a block
 //   carry     the states at the chunks' starts, one element a thread, and the span's state after its last token
 //   outputs   both terms of o, a tile of 64 tokens x 64 columns a block
@@ -53,29 +54,78 @@ __global__ void chunk_plan_kernel(const int* span_begin, int spans, int chunk, i
 }
 
 // ------------------------------------------------------------------------------------------------- prepare, scalar
-// cum[t, h]: the sum of the decays' logarithms from the chunk's first token through t; dt[t, h]. A thread a (chunk, head).
-__global__ void scalar_decay_kernel(const float* raw, int stride, const float* bias, const float* a_log, const int* chunk_begin,
-                                    float* cum, float* dt, int heads) {
+// cum[t, h]: the sum of the decays' logarithms from the chunk's first token through t; dt[t, h]. A block takes 8 heads of a
+// chunk: a warp a head, two neighbouring tokens a lane, the running sum by shuffles.
+__global__ void __launch_bounds__(256) scalar_decay_kernel(const float* raw, int stride, const float* bias, const float* a_log,
+                                                           const int* chunk_begin, float* cum, float* dt, int heads) {
+    __shared__ float raw_s[kChunk][9], cum_s[kChunk][9], dt_s[kChunk][9];
     chain_release();
     chain_wait();
-    const int h = blockIdx.x * blockDim.x + threadIdx.x;
-    if (h >= heads) return;
-    const int begin = chunk_begin[blockIdx.y], end = chunk_begin[blockIdx.y + 1];
-    const float rate = expf(a_log[h]), b = bias[h];
-    float sum = 0.0f;
-    for (int t0 = begin; t0 < end; t0 += 8) {
-        float x[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] = t0 + i < end ? raw[(size_t)(t0 + i) * stride + h] : 0.0f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            if (t0 + i >= end) break;
-            const float step = softplus_of(x[i] + b);
-            sum -= rate * step;
-            cum[(size_t)(t0 + i) * heads + h] = sum;
-            dt[(size_t)(t0 + i) * heads + h] = step;
-        }
+    const int h0 = blockIdx.x * 8;
+    const int begin = chunk_begin[blockIdx.y], count = chunk_begin[blockIdx.y + 1] - begin;
+    if (count <= 0) return;
+    for (int i = threadIdx.x; i < kChunk * 8; i += 256) {
+        const int t = i >> 3, h = i & 7;
+        raw_s[t][h] = t < count && h0 + h < heads ? raw[(size_t)(begin + t) * stride + h0 + h] : 0.0f;
     }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (h0 + warp < heads) {
+        const float rate = expf(a_log[h0 + warp]), b = bias[h0 + warp];
+        const float first = softplus_of(raw_s[2 * lane][warp] + b), second = softplus_of(raw_s[2 * lane + 1][warp] + b);
+        const float x = -rate * first, y = -rate * second;
+        float sum = x + y;
+#pragma unroll
+        for (int offset = 1; offset < 32; offset <<= 1) {
+            const float below = __shfl_up_sync(0xffffffffu, sum, offset);
+            if (lane >= offset) sum += below;
+        }
+        const float up = __shfl_up_sync(0xffffffffu, sum, 1);
+        const float before = lane > 0 ? up : 0.0f;
+        cum_s[2 * lane][warp] = before + x;
+        cum_s[2 * lane + 1][warp] = (before + x) + y;
+        dt_s[2 * lane][warp] = first;
+        dt_s[2 * lane + 1][warp] = second;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < count * 8; i += 256) {
+        const int t = i >> 3, h = i & 7;
+        if (h0 + h >= heads) continue;
+        cum[(size_t)(begin + t) * heads + h0 + h] = cum_s[t][h];
+        dt[(size_t)(begin + t) * heads + h0 + h] = dt_s[t][h];
+    }
+}
+
+// A tile of 64 x 64 floats into shared memory: rows r < rows of `src` (`stride` apart) times scale(r), columns c < columns;
+// zeros beyond. 256 threads, four neighbours a load where `four` says the rows allow it.
+template <typename Scale>
+__device__ __forceinline__ void load_tile(float (*dst)[kPitch], const float* src, long long stride, int rows, int columns,
+                                          bool four, Scale scale) {
+    if (four) {
+        float4 x[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = (threadIdx.x >> 4) + 16 * u, c = (threadIdx.x & 15) * 4;
+            x[u] = r < rows && c < columns ? *reinterpret_cast<const float4*>(src + r * stride + c)
+                                           : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = (threadIdx.x >> 4) + 16 * u, c = (threadIdx.x & 15) * 4;
+            const float f = scale(r);
+            *reinterpret_cast<float4*>(&dst[r][c]) = make_float4(x[u].x * f, x[u].y * f, x[u].z * f, x[u].w * f);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < kChunk * kChunk; i += 256) {
+        const int r = i >> 6, c = i & 63;
+        dst[r][c] = r < rows && c < columns ? src[r * stride + c] * scale(r) : 0.0f;
+    }
+}
+struct NoScale { __device__ __forceinline__ float operator()(int) const { return 1.0f; } };
+// rows that begin at multiples of four floats (every offset in them is one of `sizes`, a sum of multiples where those are)
+__device__ __forceinline__ bool by_fours(const float* p, long long stride, int sizes) {
+    return ((((unsigned long long)p >> 2) | (unsigned long long)stride | (unsigned)sizes) & 3) == 0;
 }
 
 // products[chunk, group, i, j] = q_i . k_j, 64 x 64 a block
@@ -92,14 +142,13 @@ __global__ void __launch_bounds__(256) chunk_products_kernel(const float* q, int
     float acc[4][4] = {};
     for (int e0 = 0; e0 < dim; e0 += kChunk) {
         if (e0 > 0) __syncthreads();
-        for (int i = threadIdx.x; i < kChunk * kChunk; i += 256) {
-            const int r = i >> 6, e = i & 63;
-            const bool ok = r < count && e0 + e < dim;
-            q_s[r][e] = ok ? q[(size_t)(begin + r) * q_stride + (size_t)group * dim + e0 + e] : 0.0f;
-            k_s[r][e] = ok ? k[(size_t)(begin + r) * k_stride + (size_t)group * dim + e0 + e] : 0.0f;
-        }
+        load_tile(q_s, q + (size_t)begin * q_stride + (size_t)group * dim + e0, q_stride, count, dim - e0,
+                  by_fours(q, q_stride, dim), NoScale());
+        load_tile(k_s, k + (size_t)begin * k_stride + (size_t)group * dim + e0, k_stride, count, dim - e0,
+                  by_fours(k, k_stride, dim), NoScale());
         __syncthreads();
         const int width = min(kChunk, (dim - e0 + 3) & ~3);
+#pragma unroll 1
         for (int e = 0; e < width; e += 4) {
             float4 a[4], b[4];
 #pragma unroll
@@ -131,102 +180,133 @@ struct ChannelPrepareArgs {
     int heads, dim;
 };
 
+constexpr float kLeastDecay = 1e-8f;
+constexpr int kBlock = 8, kBlocks = kChunk / kBlock;
+
+__host__ __device__ constexpr int channel_prepare_floats(int D) { return 2 * kChunk * (D + 4) + (36 + 4 * kBlocks) * D; }
+
+// D: the key size, padded to a multiple of 32
+template <int D>
 __global__ void __launch_bounds__(256) channel_prepare_kernel(const ChannelPrepareArgs p) {
-    constexpr int kSub = 16, kWarps = 8, kMost = kDecayMaxDim / 32;
+    constexpr int kPitchD = D + 4;
     extern __shared__ __align__(16) float smem[];
     chain_release();
     chain_wait();
-    const int chunk = blockIdx.y, head = blockIdx.x;
+    const int chunk = blockIdx.y, head = blockIdx.x, tid = threadIdx.x;
     const int begin = p.chunk_begin[chunk], count = p.chunk_begin[chunk + 1] - begin;
     if (count <= 0) return;
-    const int dim = p.dim, pitch = dim + 1;
-    float* q_s = smem;                       // [64][pitch]
-    float* k_s = q_s + kChunk * pitch;
-    float* a_s = k_s + kChunk * pitch;
-    float* m_s = a_s + kChunk * pitch;       // [64][65]
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int subs = (count + kSub - 1) / kSub;
-    for (int i = tid; i < subs * kSub * dim; i += 256) {
-        const int r = i / dim, e = i - r * dim;
-        const size_t t = (size_t)(begin + r);
-        const bool ok = r < count;
-        q_s[r * pitch + e] = ok ? p.q[t * p.q_stride + (size_t)head * dim + e] * p.q_scale : 0.0f;
-        k_s[r * pitch + e] = ok ? p.k[t * p.k_stride + (size_t)head * dim + e] : 0.0f;
-        a_s[r * pitch + e] = ok ? root_of_sigmoid(p.z[t * p.z_stride + (size_t)head * dim + e] + p.bias[(size_t)head * dim + e],
-                                                  p.inv_tau) : 1.0f;
-    }
-    for (int i = tid; i < kChunk * 65; i += 256) m_s[i] = 0.0f;
-    __syncthreads();
-    float through = 1.0f;                    // thread e: P(1..) of the blocks done (dim <= 256: one channel a thread)
-    for (int sub = 0; sub < subs; ++sub) {
-        const int i0 = sub * kSub, here = min(kSub, count - i0);
-        // within the block: a warp carries k_j along the tokens i >= j (q, k as they are, decays of this block)
-        for (int j = warp; j < here; j += kWarps) {
-            float w[kMost];
+    const int dim = p.dim;
+    float* q_s = smem;                       // [64][kPitchD]: queries, then at their block's middle
+    float* k_s = q_s + kChunk * kPitchD;
+    float* w_s = k_s + kChunk * kPitchD;     // [36][D]: the factor between the middles of blocks I >= J at I (I + 1) / 2 + J
+    float* upper_s = w_s + 36 * D;           // [8][D]: a block's first four decays, its last four
+    float* lower_s = upper_s + kBlocks * D;
+    float* q_to = lower_s + kBlocks * D;     // [8][D]: from the middle to the chunk's start, to its end
+    float* k_to = q_to + kBlocks * D;
+    const size_t width = (size_t)p.heads * dim;
+    // a thread a (channel, block of eight tokens)
+    for (int x = tid; x < D * kBlocks; x += 256) {
+        const int e = x % D, block = x / D, i0 = block * kBlock;
+        const bool real = e < dim;
+        const size_t column = (size_t)head * dim + e;
+        const float bias = real ? p.bias[column] : 0.0f;
+        float q[kBlock], k[kBlock], a[kBlock];
 #pragma unroll
-            for (int x = 0; x < kMost; ++x) {
-                const int e = lane + 32 * x;
-                w[x] = e < dim ? k_s[(i0 + j) * pitch + e] : 0.0f;
-            }
-            for (int i = j; i < here; ++i) {
-                float sum = 0.0f;
+        for (int i = 0; i < kBlock; ++i) {
+            const size_t t = (size_t)(begin + i0 + i);
+            const bool here = real && i0 + i < count;
+            q[i] = here ? p.q[t * p.q_stride + column] : 0.0f;
+            k[i] = here ? p.k[t * p.k_stride + column] : 0.0f;
+            a[i] = here ? p.z[t * p.z_stride + column] : 0.0f;
+        }
 #pragma unroll
-                for (int x = 0; x < kMost; ++x) {
-                    const int e = lane + 32 * x;
-                    if (e >= dim) continue;
-                    if (i > j) w[x] *= a_s[(i0 + i) * pitch + e];
-                    sum = fmaf(q_s[(i0 + i) * pitch + e], w[x], sum);
-                }
-                sum = warp_sum(sum);
-                if (lane == 0) m_s[(i0 + i) * 65 + i0 + j] = sum;
-            }
-        }
-        __syncthreads();
-        // q to the block's start, k to its end
-        float block = 1.0f;
-        if (tid < dim) {
-            for (int i = 0; i < here; ++i) {
-                block *= a_s[(i0 + i) * pitch + tid];
-                q_s[(i0 + i) * pitch + tid] *= block;
-            }
-            float after = 1.0f;
-            for (int i = here - 1; i >= 0; --i) {
-                k_s[(i0 + i) * pitch + tid] *= after;
-                after *= a_s[(i0 + i) * pitch + tid];
-            }
-        }
-        __syncthreads();
-        // against the tokens of the blocks before, whose k stands at this block's start
-        for (int x = tid; x < here * i0; x += 256) {
-            const int i = x / i0, j = x - i * i0;
-            const float* qr = q_s + (i0 + i) * pitch;
-            const float* kr = k_s + j * pitch;
-            float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            int e = 0;
-            for (; e + 4 <= dim; e += 4) {
+        for (int i = 0; i < kBlock; ++i)
+            a[i] = real && i0 + i < count ? fmaxf(root_of_sigmoid(a[i] + bias, p.inv_tau), kLeastDecay) : 1.0f;
+        float f = 1.0f;                      // P(i+1..4), tokens 4 .. 1 of the block
 #pragma unroll
-                for (int u = 0; u < 4; ++u) sum[u] = fmaf(qr[e + u], kr[e + u], sum[u]);
-            }
-            for (; e < dim; ++e) sum[0] = fmaf(qr[e], kr[e], sum[0]);
-            m_s[(i0 + i) * 65 + j] = (sum[0] + sum[1]) + (sum[2] + sum[3]);
+        for (int i = kBlock / 2 - 1; i >= 0; --i) {
+            q_s[(i0 + i) * kPitchD + e] = q[i] * p.q_scale / f;
+            k_s[(i0 + i) * kPitchD + e] = k[i] * f;
+            f *= a[i];
         }
-        __syncthreads();
-        if (tid < dim) {
-            for (int j = 0; j < i0; ++j) k_s[j * pitch + tid] *= block;
-            for (int i = 0; i < here; ++i) q_s[(i0 + i) * pitch + tid] *= through;
-            through *= block;
+        upper_s[block * D + e] = f;
+        f = 1.0f;                            // P(5..i)
+#pragma unroll
+        for (int i = kBlock / 2; i < kBlock; ++i) {
+            f *= a[i];
+            q_s[(i0 + i) * kPitchD + e] = q[i] * p.q_scale * f;
+            k_s[(i0 + i) * kPitchD + e] = k[i] / f;
         }
+        lower_s[block * D + e] = f;
     }
     __syncthreads();
-    for (int i = tid; i < count * dim; i += 256) {
-        const int r = i / dim, e = i - r * dim;
-        const size_t at = (size_t)(begin + r) * p.heads * dim + (size_t)head * dim + e;
-        p.q_out[at] = q_s[r * pitch + e];
-        p.k_out[at] = k_s[r * pitch + e];
+    for (int x = tid; x < D * kBlocks; x += 256) {
+        const int e = x % D, block = x / D;
+        float f = lower_s[block * D + e];    // from the middle of `block` to the end of the blocks so far
+        w_s[(block * (block + 1) / 2 + block) * D + e] = 1.0f;
+        for (int later = block + 1; later < kBlocks; ++later) {
+            w_s[(later * (later + 1) / 2 + block) * D + e] = f * upper_s[later * D + e];
+            f *= upper_s[later * D + e] * lower_s[later * D + e];
+        }
+        k_to[block * D + e] = f;
+        float g = upper_s[block * D + e];
+        for (int earlier = 0; earlier < block; ++earlier) g *= upper_s[earlier * D + e] * lower_s[earlier * D + e];
+        q_to[block * D + e] = g;
+        if (block == 0 && e < dim) p.total[(size_t)chunk * width + (size_t)head * dim + e] = f * upper_s[e];
     }
-    if (tid < dim) p.total[(size_t)chunk * p.heads * dim + (size_t)head * dim + tid] = through;
+    __syncthreads();
+    const int tx = tid & 15, ty = tid >> 4;
+    float acc[4][4] = {};
+    {
+        // tokens ty * 4 + i (block I, the warp's number) against tokens tx + 16 j (blocks 2 j and 2 j + 1, none beyond I)
+        const int own = ty >> 1;
+        const float* w[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j] = w_s + (own * (own + 1) / 2 + min((tx >> 3) + 2 * j, own)) * D;
+#pragma unroll 1
+        for (int e = 0; e < ((dim + 3) & ~3); e += 4) {
+            float4 a[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const float4*>(q_s + (ty * 4 + i) * kPitchD + e);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (2 * j > own) continue;
+                const float4 f = *reinterpret_cast<const float4*>(w[j] + e);
+                float4 b = *reinterpret_cast<const float4*>(k_s + (tx + 16 * j) * kPitchD + e);
+                b.x *= f.x; b.y *= f.y; b.z *= f.z; b.w *= f.w;
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    acc[i][j] = fmaf(a[i].x, b.x, fmaf(a[i].y, b.y, fmaf(a[i].z, b.z, fmaf(a[i].w, b.w, acc[i][j]))));
+            }
+        }
+    }
     float* dst = p.products + ((size_t)chunk * p.heads + head) * kChunk * kChunk;
-    for (int i = tid; i < kChunk * kChunk; i += 256) dst[i] = m_s[(i >> 6) * 65 + (i & 63)];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            dst[(ty * 4 + i) * kChunk + tx + 16 * j] = tx + 16 * j <= ty * 4 + i ? acc[i][j] : 0.0f;
+    for (int x = tid; x < count * D; x += 256) {
+        const int r = x / D, e = x % D;
+        if (e >= dim) continue;
+        const size_t at = (size_t)(begin + r) * width + (size_t)head * dim + e;
+        p.q_out[at] = q_s[r * kPitchD + e] * q_to[(r >> 3) * D + e];
+        p.k_out[at] = k_s[r * kPitchD + e] * k_to[(r >> 3) * D + e];
+    }
+}
+
+template <int D>
+static int launch_channel_prepare(const ChannelPrepareArgs& args, int chunks, cudaStream_t stream) {
+    constexpr size_t smem = (size_t)channel_prepare_floats(D) * sizeof(float);
+    if (smem > 40 * 1024) {
+        const cudaError_t status = cudaFuncSetAttribute(channel_prepare_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (status != cudaSuccess) {
+            set_error("channel_decay_scan: %s", cudaGetErrorString(status));
+            return -2;
+        }
+    }
+    launch_chained(channel_prepare_kernel<D>, dim3(args.heads, chunks), 256, smem, stream, args);
+    return check_launch("channel_prepare");
 }
 
 // --------------------------------------------------------------------------------------------- states, carry, outputs
@@ -264,12 +344,12 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs p) {
         }
         __syncthreads();
     }
-    for (int i = threadIdx.x; i < count * kChunk; i += 256) {
-        const int r = i >> 6, c = i & 63;
-        const float x = e0 + c < p.dim ? p.k[(size_t)(begin + r) * p.k_stride + k_at + c] : 0.0f;
-        k_s[r][c] = CHANNEL ? x : x * w_s[r];
-        v_s[r][c] = c0 + c < p.vdim ? p.v[(size_t)(begin + r) * p.v_stride + (size_t)head * p.vdim + c0 + c] : 0.0f;
-    }
+    const float* k_src = p.k + (size_t)begin * p.k_stride + k_at;
+    if (CHANNEL) load_tile(k_s, k_src, p.k_stride, count, p.dim - e0, by_fours(p.k, p.k_stride, p.dim), NoScale());
+    else load_tile(k_s, k_src, p.k_stride, count, p.dim - e0, by_fours(p.k, p.k_stride, p.dim),
+                   [&](int r) { return r < count ? w_s[r] : 0.0f; });
+    load_tile(v_s, p.v + (size_t)begin * p.v_stride + (size_t)head * p.vdim + c0, p.v_stride, count, p.vdim - c0,
+              by_fours(p.v, p.v_stride, p.vdim), NoScale());
     __syncthreads();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float acc[4][4] = {};
@@ -284,10 +364,16 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs p) {
             for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
     }
     float* dst = p.states + ((size_t)chunk * p.heads + head) * p.dim * p.vdim;
+    const bool four = (p.vdim & 3) == 0;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int e = e0 + ty * 4 + i;
         if (e >= p.dim) continue;
+        if (four) {
+            if (c0 + tx * 4 < p.vdim)
+                *reinterpret_cast<float4*>(dst + (size_t)e * p.vdim + c0 + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int c = c0 + tx * 4 + j;
@@ -296,45 +382,65 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs p) {
     }
 }
 
-// a thread an element of the state: a chunk's own sum is replaced by the state before the chunk
-template <bool CHANNEL>
-__global__ void chunk_carry_kernel(const ChunkArgs p, float* state, long long slot_stride, const int* span_slot,
-                                   const int* span_first) {
+// a thread V neighbouring elements of the state: a chunk's own sum is replaced by the state before the chunk
+template <bool CHANNEL, int V>
+__global__ void __launch_bounds__(128) chunk_carry_kernel(const ChunkArgs p, float* state, long long slot_stride,
+                                                          const int* span_slot, const int* span_first) {
     chain_release();
     chain_wait();
     const int elements = p.heads * p.dim * p.vdim;
-    const int e = blockIdx.x * blockDim.x + threadIdx.x;
+    const int e = (blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (e >= elements) return;
     const int span = blockIdx.y;
     const int first = span_first[span], last = span_first[span + 1];
     if (first == last) return;
-    const int row = e / p.vdim, head = row / p.dim;                    // row: head * dim + key channel
+    const int row = e / p.vdim, head = row / p.dim;                    // row: head * dim + key channel (V divides vdim)
     float* cell = state + (long long)span_slot[span] * slot_stride + e;
-    float s = *cell;
-    constexpr int kAhead = 4;
+    float s[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) s[i] = cell[i];
+    constexpr int kAhead = 8;
     for (int c0 = first; c0 < last; c0 += kAhead) {
-        float own[kAhead], keep[kAhead];
+        float own[kAhead][V], keep[kAhead];
+        int ends[kAhead];
 #pragma unroll
         for (int i = 0; i < kAhead; ++i) {
             const int c = c0 + i;
             if (c >= last) continue;
-            own[i] = p.states[(size_t)c * elements + e];
-            keep[i] = CHANNEL ? p.total[(size_t)c * p.heads * p.dim + row]
-                              : p.cum[(size_t)(p.chunk_begin[c + 1] - 1) * p.heads + head];
+            ends[i] = CHANNEL ? 0 : p.chunk_begin[c + 1] - 1;
+            const float* src = p.states + (size_t)c * elements + e;
+            if (V == 4) {
+                const float4 x = *reinterpret_cast<const float4*>(src);
+                own[i][0] = x.x; own[i][1 % V] = x.y; own[i][2 % V] = x.z; own[i][3 % V] = x.w;
+            } else {
+                own[i][0] = *src;
+            }
+            if (CHANNEL) keep[i] = p.total[(size_t)c * p.heads * p.dim + row];
+        }
+        if (!CHANNEL) {
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i)
+                if (c0 + i < last) keep[i] = p.cum[(size_t)ends[i] * p.heads + head];
         }
 #pragma unroll
         for (int i = 0; i < kAhead; ++i) {
             const int c = c0 + i;
             if (c >= last) continue;
-            p.states[(size_t)c * elements + e] = s;
-            s = fmaf(CHANNEL ? keep[i] : expf(keep[i]), s, own[i]);
+            float* dst = p.states + (size_t)c * elements + e;
+            if (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(s[0], s[1 % V], s[2 % V], s[3 % V]);
+            else *dst = s[0];
+            const float f = CHANNEL ? keep[i] : expf(keep[i]);
+#pragma unroll
+            for (int j = 0; j < V; ++j) s[j] = fmaf(f, s[j], own[i][j]);
         }
     }
-    *cell = s;
+#pragma unroll
+    for (int i = 0; i < V; ++i) cell[i] = s[i];
 }
 
 __device__ __forceinline__ void tile_product(const float (*a_s)[kPitch], const float (*b_s)[kPitch], int depth, int tx, int ty,
                                              float (&acc)[4][4]) {
+#pragma unroll 1
     for (int k = 0; k < depth; k += 4) {
         float4 a[4], b[4];
 #pragma unroll
@@ -356,7 +462,7 @@ __device__ __forceinline__ void tile_product(const float (*a_s)[kPitch], const f
 }
 
 template <bool CHANNEL>
-__global__ void __launch_bounds__(256) chunk_outputs_kernel(const ChunkArgs p) {
+__global__ void __launch_bounds__(256, 4) chunk_outputs_kernel(const ChunkArgs p) {
     __shared__ __align__(16) float a_s[kChunk][kPitch];
     __shared__ __align__(16) float b_s[kChunk][kPitch];
     __shared__ float cum_s[kChunk], dt_s[kChunk];
@@ -376,12 +482,24 @@ __global__ void __launch_bounds__(256) chunk_outputs_kernel(const ChunkArgs p) {
     }
     // the chunk's own tokens
     const float* m = p.products + ((size_t)chunk * (CHANNEL ? p.heads : p.groups) + group) * kChunk * kChunk;
-    for (int i = threadIdx.x; i < kChunk * kChunk; i += 256) {
-        const int r = i >> 6, c = i & 63;
-        float x = 0.0f;
-        if (c <= r && r < count) x = CHANNEL ? m[i] : m[i] * expf(cum_s[r] - cum_s[c]) * dt_s[c];
-        a_s[r][c] = x;
-        b_s[r][c] = r < count && c0 + c < p.vdim ? p.v[(size_t)(begin + r) * p.v_stride + (size_t)head * p.vdim + c0 + c] : 0.0f;
+    load_tile(b_s, p.v + (size_t)begin * p.v_stride + (size_t)head * p.vdim + c0, p.v_stride, count, p.vdim - c0,
+              by_fours(p.v, p.v_stride, p.vdim), NoScale());
+    {
+        float4 x[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) x[u] = reinterpret_cast<const float4*>(m)[threadIdx.x + 256 * u];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = (threadIdx.x >> 4) + 16 * u, c = (threadIdx.x & 15) * 4;
+            float v[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const bool seen = c + i <= r && r < count;
+                if (CHANNEL) v[i] = seen ? v[i] : 0.0f;
+                else v[i] = seen ? v[i] * expf(cum_s[r] - cum_s[c + i]) * dt_s[c + i] : 0.0f;
+            }
+            *reinterpret_cast<float4*>(&a_s[r][c]) = make_float4(v[0], v[1], v[2], v[3]);
+        }
     }
     __syncthreads();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -398,16 +516,12 @@ __global__ void __launch_bounds__(256) chunk_outputs_kernel(const ChunkArgs p) {
     const float* state = p.states + ((size_t)chunk * p.heads + head) * p.dim * p.vdim;
     for (int e0 = 0; e0 < p.dim; e0 += kChunk) {
         __syncthreads();
-        for (int i = threadIdx.x; i < kChunk * kChunk; i += 256) {
-            const int r = i >> 6, c = i & 63;
-            float x = 0.0f;
-            if (r < count && e0 + c < p.dim) {
-                x = p.q[(size_t)(begin + r) * p.q_stride + (size_t)group * p.dim + e0 + c];
-                if (!CHANNEL) x *= expf(cum_s[r]);
-            }
-            a_s[r][c] = x;
-            b_s[r][c] = e0 + r < p.dim && c0 + c < p.vdim ? state[(size_t)(e0 + r) * p.vdim + c0 + c] : 0.0f;
-        }
+        const float* q_src = p.q + (size_t)begin * p.q_stride + (size_t)group * p.dim + e0;
+        if (CHANNEL) load_tile(a_s, q_src, p.q_stride, count, p.dim - e0, by_fours(p.q, p.q_stride, p.dim), NoScale());
+        else load_tile(a_s, q_src, p.q_stride, count, p.dim - e0, by_fours(p.q, p.q_stride, p.dim),
+                       [&](int r) { return expf(cum_s[r]); });
+        load_tile(b_s, state + (size_t)e0 * p.vdim + c0, p.vdim, p.dim - e0, p.vdim - c0, by_fours(p.states, p.vdim, p.dim * p.vdim),
+                  NoScale());
         __syncthreads();
         tile_product(a_s, b_s, min(kChunk, (p.dim - e0 + 3) & ~3), tx, ty, acc);
     }
@@ -416,6 +530,10 @@ __global__ void __launch_bounds__(256) chunk_outputs_kernel(const ChunkArgs p) {
         const int r = ty * 4 + i;
         if (r >= count) continue;
         float* dst = p.out + (size_t)(begin + r) * p.heads * p.vdim + (size_t)head * p.vdim + c0;
+        if ((p.vdim & 3) == 0) {
+            if (c0 + tx * 4 < p.vdim) *reinterpret_cast<float4*>(dst + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j)
             if (c0 + tx * 4 + j < p.vdim) dst[tx * 4 + j] = acc[i][j];
@@ -575,8 +693,12 @@ static int launch_chunks(const ChunkArgs& p, float* state, long long slot_stride
     int status = check_launch("chunk_states");
     if (status != 0) return status;
     const long long elements = (long long)p.heads * p.dim * p.vdim;
-    launch_chained(chunk_carry_kernel<CHANNEL>, dim3((unsigned)((elements + 255) / 256), spans), 256, 0, stream, p, state,
-                   slot_stride, span_slot, span_first);
+    if (p.vdim % 4 == 0)                     // (scratch and slots are laid out for 16-byte accesses)
+        launch_chained(chunk_carry_kernel<CHANNEL, 4>, dim3((unsigned)((elements / 4 + 127) / 128), spans), 128, 0, stream, p, state,
+                       slot_stride, span_slot, span_first);
+    else
+        launch_chained(chunk_carry_kernel<CHANNEL, 1>, dim3((unsigned)((elements + 127) / 128), spans), 128, 0, stream, p, state,
+                       slot_stride, span_slot, span_first);
     status = check_launch("chunk_carry");
     if (status != 0) return status;
     launch_chained(chunk_outputs_kernel<CHANNEL>, dim3(v_tiles, p.heads, chunks), 256, 0, stream, p);
@@ -613,16 +735,10 @@ CELEG_API int celeg_channel_decay_scan(const float* q, int q_stride, const float
     const int* span_first = plan + max_chunks + 1;
     const ChannelPrepareArgs first = {q, q_stride, k, k_stride, z, z_stride, bias, inv_tau, q_scale, plan, q_out, k_out, total,
                                       products, heads, dim};
-    const size_t smem = ((size_t)3 * kChunk * (dim + 1) + kChunk * 65) * sizeof(float);
-    if (smem > 40 * 1024) {
-        const cudaError_t status = cudaFuncSetAttribute(channel_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (status != cudaSuccess) {
-            set_error("channel_decay_scan: %s", cudaGetErrorString(status));
-            return -2;
-        }
-    }
-    launch_chained(channel_prepare_kernel, dim3(heads, chunks), 256, smem, stream, first);
-    const int status = check_launch("channel_prepare");
+    const int status = dim <= 32 ? launch_channel_prepare<32>(first, chunks, stream)
+                     : dim <= 64 ? launch_channel_prepare<64>(first, chunks, stream)
+                     : dim <= 128 ? launch_channel_prepare<128>(first, chunks, stream)
+                                  : launch_channel_prepare<256>(first, chunks, stream);
     if (status != 0) return status;
     const ChunkArgs p = {q_out, heads * dim, k_out, heads * dim, v, v_stride, nullptr, nullptr, total, products, nullptr, plan,
                          states, out, heads, heads, dim, vdim};
@@ -643,7 +759,7 @@ CELEG_API int celeg_scalar_decay_scan(const float* q, int q_stride, const float*
                   "scalar_decay_scan: %d chunks of %d, %d spans or %d heads exceed one launch", chunks, max_chunks, spans, heads);
     if (spans == 0 || chunks == 0) return 0;
     const int* span_first = plan + max_chunks + 1;
-    launch_chained(scalar_decay_kernel, dim3((heads + 63) / 64, chunks), 64, 0, stream, raw, raw_stride, dt_bias, a_log, plan,
+    launch_chained(scalar_decay_kernel, dim3((heads + 7) / 8, chunks), 256, 0, stream, raw, raw_stride, dt_bias, a_log, plan,
                    cum, dt, heads);
     int status = check_launch("scalar_decay");
     if (status != 0) return status;

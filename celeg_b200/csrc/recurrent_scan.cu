@@ -445,6 +445,67 @@ __global__ void gated_head_norm_pairs_kernel(const float* o, const float* gate, 
     }
 }
 
+// The same for units of 129 to 1,024 entries, four neighbours a lane and access: a warp a unit, everything in registers
+// between the sum and the result. Q: quads a lane.
+template <typename A, int Q>
+__global__ void __launch_bounds__(128) gated_unit_norm_kernel(const float* o, const float* gate, int gate_stride,
+                                                              const float* weight, int weight_per_head, A* out, int tokens,
+                                                              int heads, int vdim, float eps, int gate_kind) {
+    chain_release();
+    chain_wait();
+    const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= (long long)tokens * heads) return;
+    const int lane = threadIdx.x & 31;
+    const int t = (int)(unit / heads), h = (int)(unit % heads);
+    const float4* src = reinterpret_cast<const float4*>(o + ((size_t)t * heads + h) * vdim);
+    const float4* g = reinterpret_cast<const float4*>(gate + (size_t)t * gate_stride + (size_t)h * vdim);
+    const float4* w = reinterpret_cast<const float4*>(weight ? weight + (weight_per_head ? (size_t)h * vdim : 0) : nullptr);
+    const int quads = vdim >> 2;
+    float4 x[Q], z[Q];
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+        const int i = lane + 32 * u;
+        x[u] = i < quads ? src[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        z[u] = i < quads ? g[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    float sum = 0.0f;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+        z[u] = make_float4(output_gate(z[u].x, gate_kind), output_gate(z[u].y, gate_kind), output_gate(z[u].z, gate_kind),
+                           output_gate(z[u].w, gate_kind));
+        if (gate_kind >= 2) { x[u].x *= z[u].x; x[u].y *= z[u].y; x[u].z *= z[u].z; x[u].w *= z[u].w; }
+        sum += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)vdim + eps);
+    A* dst = out + ((size_t)t * heads + h) * vdim;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+        const int i = lane + 32 * u;
+        if (i >= quads) continue;
+        const float4 s = w ? __ldg(w + i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+        float4 y = make_float4(x[u].x * inv * s.x, x[u].y * inv * s.y, x[u].z * inv * s.z, x[u].w * inv * s.w);
+        if (gate_kind < 2) { y.x *= z[u].x; y.y *= z[u].y; y.z *= z[u].z; y.w *= z[u].w; }
+        if (sizeof(A) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(y.x, y.y), hi = __floats2bfloat162_rn(y.z, y.w);
+            uint2 raw;
+            raw.x = *reinterpret_cast<const unsigned*>(&lo);
+            raw.y = *reinterpret_cast<const unsigned*>(&hi);
+            *reinterpret_cast<uint2*>(dst + 4 * i) = raw;
+        } else {
+            *reinterpret_cast<float4*>(dst + 4 * i) = y;
+        }
+    }
+}
+
+template <typename A>
+static void launch_unit_norm(const float* o, const float* gate, int gate_stride, const float* weight, int weight_per_head,
+                             A* out, int tokens, int heads, int vdim, float eps, int gate_kind, cudaStream_t stream) {
+    const unsigned blocks = (unsigned)(((long long)tokens * heads + 3) / 4);
+    auto kernel = vdim <= 256 ? gated_unit_norm_kernel<A, 2> : vdim <= 512 ? gated_unit_norm_kernel<A, 4> : gated_unit_norm_kernel<A, 8>;
+    launch_chained(kernel, blocks, 128, 0, stream, o, gate, gate_stride, weight, weight_per_head, out, tokens, heads, vdim, eps,
+                   gate_kind);
+}
+
 // The same for wide units (one norm over all heads' columns together): a block per (token, head), 16-byte reads
 // where the rows allow them. The order of the sum differs from the warp's; both are float32 sums of the same squares.
 template <typename A>
@@ -1030,6 +1091,16 @@ CELEG_API int celeg_gated_head_norm(const float* o, const float* gate, int gate_
                   gate_kind);
     if (tokens == 0) return 0;
     const long long units = (long long)tokens * heads;
+    if (vdim > 128 && vdim <= 1024 && units >= 2048 && vdim % 4 == 0 && gate_stride % 4 == 0 &&
+        (act_dtype == kFloat32 || act_dtype == kBFloat16) &&
+        (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0) {
+        if (act_dtype == kFloat32)
+            launch_unit_norm<float>(o, gate, gate_stride, weight, weight_per_head, (float*)out, tokens, heads, vdim, eps, gate_kind, stream);
+        else
+            launch_unit_norm<__nv_bfloat16>(o, gate, gate_stride, weight, weight_per_head, (__nv_bfloat16*)out, tokens, heads, vdim,
+                                            eps, gate_kind, stream);
+        return check_launch("gated_head_norm");
+    }
     if (vdim >= 512) {          // a unit is worth a block
         CELEG_REQUIRE(units <= 0x7fffffffLL, "gated_head_norm: %lld units exceed one launch", units);
         const int vectors = vdim % 4 == 0 && gate_stride % 4 == 0 && ((uintptr_t)o | (uintptr_t)gate | (uintptr_t)weight) % 16 == 0;
