@@ -209,11 +209,13 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
     const float* row = p.proj + (size_t)t * p.proj_stride;
     float c[E], s[E];
     const int units = p.q_heads + 2 * p.kv_heads;
-    for (int base = warp; base < units; base += kAhead * warps) {
+    // (few tokens: several blocks share a token's heads)
+    const int first = (blockIdx.y * warps + warp), step = gridDim.y * warps;
+    for (int base = first; base < units; base += kAhead * step) {
         float2 v[kAhead][E];
 #pragma unroll
         for (int a = 0; a < kAhead; ++a) {
-            const int unit = base + a * warps;
+            const int unit = base + a * step;
             const bool value = unit >= p.q_heads + p.kv_heads;
             const int at = value ? qk_width + (unit - p.q_heads - p.kv_heads) * p.value_dim : unit * p.head_dim;
 #pragma unroll
@@ -230,7 +232,7 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
                 }
             }
         }
-        if (base == warp) {                                // (the angles, while the first heads are on their way)
+        if (base == first) {                               // (the angles, while the first heads are on their way)
 #pragma unroll
             for (int x = 0; x < E; ++x) {
                 c[x] = 1.0f;
@@ -245,7 +247,7 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
         }
 #pragma unroll
         for (int a = 0; a < kAhead; ++a) {
-            const int unit = base + a * warps;
+            const int unit = base + a * step;
             if (unit >= units) continue;                   // (the same for the whole warp)
             const bool is_q = unit < p.q_heads, value = unit >= p.q_heads + p.kv_heads;
             const int size = value ? p.value_dim : p.head_dim;
@@ -288,8 +290,12 @@ __global__ void __launch_bounds__(128) qkv_prepare_heads_kernel(const QkvPrepare
 template <typename A>
 static void launch_prepare_heads(const QkvPrepareArgs& args, int tokens, cudaStream_t stream) {
     const int size = args.head_dim > args.value_dim ? args.head_dim : args.value_dim;
-    if (size <= 64) launch_chained(qkv_prepare_heads_kernel<A, 1>, tokens, 128, 0, stream, args);
-    else launch_chained(qkv_prepare_heads_kernel<A, 2>, tokens, 128, 0, stream, args);
+    const int units = args.q_heads + 2 * args.kv_heads;
+    int share = tokens < 148 ? (148 + tokens - 1) / tokens : 1;      // blocks that share a token, four heads each at least
+    if (share > (units + 3) / 4) share = (units + 3) / 4;
+    const dim3 grid(tokens, share);
+    if (size <= 64) launch_chained(qkv_prepare_heads_kernel<A, 1>, grid, 128, 0, stream, args);
+    else launch_chained(qkv_prepare_heads_kernel<A, 2>, grid, 128, 0, stream, args);
 }
 
 }  // namespace celeg_b200
@@ -354,7 +360,8 @@ CELEG_API int celeg_qkv_prepare(const float* proj, int proj_stride, const float*
     }
     // A block's time is a chain of dependent loads (position, span, page) and two passes over a short row: more and
     // smaller blocks an SM hide it better than wide ones (2,048 tokens of 16 + 4 heads of 64: 20 us with 256 threads).
-    const int threads = (q_heads + kv_heads) * head_dim <= 4096 ? 128 : 256;
+    // (few tokens: nothing else hides it, so a block is as wide as its row allows)
+    const int threads = tokens <= 148 ? 512 : (q_heads + kv_heads) * head_dim <= 4096 ? 128 : 256;
     if (act_dtype == kFloat32)
         launch_chained(qkv_prepare_kernel<float>, tokens, threads, smem, stream, args);
     else

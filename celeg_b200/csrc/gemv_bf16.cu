@@ -33,7 +33,8 @@ namespace celeg_b200 {
 constexpr int kGemvMaxConvTaps = 16;
 
 enum GemvMode : int { kGemvStoreBf16 = 0, kGemvStoreF32 = 1, kGemvAddResidual = 2, kGemvSwiGlu = 3, kGemvConv = 4,
-                      kGemvActivation = 5 };     // y bfloat16 = act(x w^T); which activation travels in the `taps` argument
+                      kGemvActivation = 5,       // y bfloat16 = act(x w^T); which activation travels in the `taps` argument
+                      kGemvHyper = 6 };          // mixed into several residual streams (GemvHyperArgs)
 // (kGemvSwiglu: `taps` = 1 + a code of activate(), or of the clamped form, names another function of the gate than SiLU;
 // 0: SiLU)
 
@@ -65,6 +66,19 @@ struct GemvNormArgs {
     int ldxw;
     float* sumsq_out;            // [m][sumsq_out_stride], entry blockIdx.x
     int sumsq_out_stride;
+};
+
+// Several residual streams in place of one (hyper_connections.cu): the product that ends a sublayer is mixed into all of
+// them, x_t <- sum_s mix[s, t] x_s + give[t] y, and the norm of the next sublayer's weighted sum u = sum_t take[t] x_t is
+// prepared as in the add-residual mode (GemvNormArgs: x' = bf16(u * w), the sums of u^2).
+constexpr int kGemvMaxStreams = 4;
+struct GemvHyperArgs {
+    const float* single;         // [m, n]: every old stream is this row, or null
+    float* streams;              // [m, count, n]
+    int count;
+    const float* mix;            // [count, count] from, to
+    const float* give;
+    const float* take;           // or null: the plain sum
 };
 
 __device__ __forceinline__ uint4 ldg_stream(const void* ptr) {
@@ -106,11 +120,12 @@ template <int MT, int WT, int MODE, int kGemvUnroll, int kGemvWarps>
 __global__ void __launch_bounds__(kGemvWarps * 32)
 gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restrict__ w, int ldw,
                  void* __restrict__ y, int ldy, int m, int n, int k, int second_tile_offset, GemvConvArgs conv,
-                 GemvNormArgs norm, GemvPrefetch ahead) {
+                 GemvNormArgs norm, GemvPrefetch ahead, GemvHyperArgs hyper) {
     constexpr int kGemvThreads = kGemvWarps * 32;
     extern __shared__ __align__(16) float partial_raw[];
     __shared__ float row_scale[16];
     __shared__ float squares[16][17];
+    __shared__ float hyper_w[MODE == kGemvHyper ? kGemvMaxStreams * (kGemvMaxStreams + 2) : 1];      // mix | give | take
     float (*partial)[WT][MT][32][4] = reinterpret_cast<float (*)[WT][MT][32][4]>(partial_raw);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, c = lane & 3;
@@ -149,14 +164,30 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
     const bool early = MODE == kGemvConv && conv.taps <= kEarlyTaps && (int)threadIdx.x < MT * 128;
     // The epilogue that adds to the residual stream likewise: the stream's old value and the next norm's weight.
     float early_residual = 0.0f, early_next_w = 0.0f;
-    const bool early_add = MODE == kGemvAddResidual && (int)threadIdx.x < MT * 128;
+    float early_stream[MODE == kGemvHyper ? kGemvMaxStreams : 1];
+    const bool early_add = (MODE == kGemvAddResidual || MODE == kGemvHyper) && (int)threadIdx.x < MT * 128;
+    if (MODE == kGemvHyper) {                        // (constant data)
+        const int n2 = hyper.count * hyper.count;
+        for (int i = threadIdx.x; i < n2 + 2 * hyper.count; i += kGemvThreads)
+            hyper_w[i] = i < n2 ? hyper.mix[i] : i < n2 + hyper.count ? hyper.give[i - n2]
+                       : hyper.take ? hyper.take[i - n2 - hyper.count] : 1.0f;
+    }
+    auto stream_at = [&](int row, int s, int col) {
+        return hyper.single ? hyper.single + (size_t)row * n + col : hyper.streams + ((size_t)row * hyper.count + s) * n + col;
+    };
     auto fetch_early = [&]() {
         if (early_add) {
             const int i = threadIdx.x, j = i / 128, ln = (i % 128) / 4, e = i % 4;
             const int out_col = row0 + (ln >> 2) + ((e >> 1) << 3);
             const int out_row = j * 8 + ((ln & 3) << 1) + (e & 1);
             if (out_row < m && out_col < n) {
-                early_residual = reinterpret_cast<const float*>(y)[(size_t)out_row * ldy + out_col];
+                if (MODE == kGemvHyper) {
+#pragma unroll
+                    for (int s = 0; s < kGemvMaxStreams; ++s)
+                        if (s < hyper.count) early_stream[MODE == kGemvHyper ? s : 0] = *stream_at(out_row, s, out_col);
+                } else {
+                    early_residual = reinterpret_cast<const float*>(y)[(size_t)out_row * ldy + out_col];
+                }
                 if (norm.next_w) early_next_w = norm.next_w[out_col];
             }
         }
@@ -298,7 +329,7 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
         // accumulator element e of lane ln: weight row (ln/4) + 8*(e/2), activation row 2*(ln%4) + (e%2)
         const int out_col = row0 + (ln >> 2) + ((e >> 1) << 3);
         const int out_row = j * 8 + ((ln & 3) << 1) + (e & 1);
-        if (MODE == kGemvAddResidual && norm.next_w && out_row < m && out_col >= n)
+        if ((MODE == kGemvAddResidual || MODE == kGemvHyper) && norm.next_w && out_row < m && out_col >= n)
             squares[out_row][out_col - row0] = 0.0f;
         if (out_row >= m || out_col >= n) continue;
         if (norm.sumsq_in) {
@@ -325,6 +356,28 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
                 norm.xw_out[(size_t)out_row * norm.ldxw + out_col] = __float2bfloat16_rn(updated * next_w);
                 squares[out_row][out_col - row0] = updated * updated;
             }
+        } else if (MODE == kGemvHyper) {
+            const bool fetched = early_add && i == (int)threadIdx.x;
+            float x[kGemvMaxStreams];
+#pragma unroll
+            for (int s = 0; s < kGemvMaxStreams; ++s)
+                x[s] = s < hyper.count ? (fetched ? early_stream[MODE == kGemvHyper ? s : 0] : *stream_at(out_row, s, out_col)) : 0.0f;
+            const float* give = hyper_w + hyper.count * hyper.count;
+            const float* take = give + hyper.count;
+            float u = 0.0f;
+#pragma unroll
+            for (int to = 0; to < kGemvMaxStreams; ++to) {
+                if (to >= hyper.count) continue;
+                float v = give[to] * sum[0];
+#pragma unroll
+                for (int s = 0; s < kGemvMaxStreams; ++s)
+                    if (s < hyper.count) v = fmaf(hyper_w[s * hyper.count + to], x[s], v);
+                hyper.streams[((size_t)out_row * hyper.count + to) * n + out_col] = v;
+                u = fmaf(take[to], v, u);
+            }
+            const float next_w = fetched ? early_next_w : norm.next_w[out_col];
+            norm.xw_out[(size_t)out_row * norm.ldxw + out_col] = __float2bfloat16_rn(u * next_w);
+            squares[out_row][out_col - row0] = u * u;
         } else if (MODE == kGemvConv) {
             // B, C, X as a plain product would store them (one rounding each), then the span kernel's
             // arithmetic in the same order, so that both ways give the same bits
@@ -367,7 +420,7 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
                 __float2bfloat16_rn(conv.taps > 0 ? gated_value(gate, up, conv.taps - 1, conv.gate) : gate / (1.0f + expf(-gate)) * up);
         }
     }
-    if (MODE == kGemvAddResidual && norm.next_w) {
+    if ((MODE == kGemvAddResidual || MODE == kGemvHyper) && norm.next_w) {
         // this block's 16 columns of every row, summed in a fixed order
         __syncthreads();
         if (threadIdx.x < m) {
@@ -380,6 +433,7 @@ gemv_bf16_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restric
 }
 
 static thread_local GemvPrefetch g_gemv_ahead = {nullptr, 0};      // the caller's hint for the next product (taken at its entry)
+static thread_local GemvHyperArgs g_gemv_hyper = {};      // of the product being launched
 static thread_local GemvPrefetch g_gemv_launch_ahead = {nullptr, 0};   // the hint of the product being launched
 
 template <int MT, int WT, int MODE, int UNROLL, int WARPS>
@@ -398,7 +452,7 @@ static int launch_one(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* w, i
     const GemvPrefetch ahead = g_gemv_launch_ahead;
     g_gemv_launch_ahead = {nullptr, 0};
     launch_chained_class(kChainGemv, kernel, (n + 15) / 16, WARPS * 32, smem, stream, x, ldx, w, ldw, y, ldy, m, n, k,
-                         tile_offset, conv, norm, ahead);
+                         tile_offset, conv, norm, ahead, g_gemv_hyper);
     return check_launch("gemv_bf16");
 }
 
@@ -414,6 +468,8 @@ static int launch_gemv(int mode, const __nv_bfloat16* x, int ldx, const __nv_bfl
             return launch_one<MT, 1, kGemvActivation, UNROLL, WARPS>(x, ldx, w, ldw, y, ldy, m, n, k, 0, conv, norm, stream);
         case kGemvAddResidual:
             return launch_one<MT, 1, kGemvAddResidual, UNROLL, WARPS>(x, ldx, w, ldw, y, ldy, m, n, k, 0, conv, norm, stream);
+        case kGemvHyper:
+            return launch_one<MT, 1, kGemvHyper, UNROLL, WARPS>(x, ldx, w, ldw, y, ldy, m, n, k, 0, conv, norm, stream);
         case kGemvSwiGlu:
             // n = inner width; rows [0, n) are the gate, rows [n, 2n) the up projection
             // (9 to 16 rows: half the loads in flight per warp, or the registers allow one block per SM only)
@@ -533,4 +589,27 @@ CELEG_API int celeg_gemv_bf16_split_norm(const void* x, int ldx, const void* w, 
     const GemvNormArgs norm = {sumsq_in, partials_in, sumsq_in_stride, eps, width,
                                next_w, (__nv_bfloat16*)xw_out, ldxw, sumsq_out, sumsq_out_stride};
     return gemv_checked(x, ldx, w, ldw, y, ldy, m, n, k, mode, conv_w, taps, state, slot_stride, span_slot, norm, stream);
+}
+
+// The product that ends a sublayer, mixed into `count` residual streams (float32 [m, count, n]; single, [m, n]: every old
+// stream is this row, or null), and the next sublayer's norm prepared: see GemvHyperArgs and celeg_gemv_bf16_split_norm
+// (sumsq_in null: x is as it is).
+CELEG_API int celeg_gemv_hyper(const void* x, int ldx, const void* w, int ldw, int m, int n, int k, const float* single,
+                               float* streams, int count, const float* mix, const float* give, const float* take,
+                               const float* sumsq_in, int partials_in, int sumsq_in_stride, float eps, int width,
+                               const float* next_w, void* xw_out, int ldxw, float* sumsq_out, int sumsq_out_stride,
+                               cudaStream_t stream) {
+    CELEG_REQUIRE(count >= 1 && count <= kGemvMaxStreams && streams && mix && give,
+                  "gemv_hyper: %d streams (1 to %d) with their weights", count, kGemvMaxStreams);
+    CELEG_REQUIRE(!sumsq_in || (partials_in > 0 && sumsq_in_stride >= partials_in && eps > 0.0f && width > 0),
+                  "gemv_hyper: the row scale needs partials_in=%d <= stride=%d, eps > 0 and a width", partials_in, sumsq_in_stride);
+    CELEG_REQUIRE(next_w && xw_out && sumsq_out && ldxw >= n && sumsq_out_stride >= (n + 15) / 16,
+                  "gemv_hyper: the norm that follows needs outputs of ldxw=%d >= n=%d and a stride of at least %d sums", ldxw, n,
+                  (n + 15) / 16);
+    const GemvNormArgs norm = {sumsq_in, partials_in, sumsq_in_stride, eps, width,
+                               next_w, (__nv_bfloat16*)xw_out, ldxw, sumsq_out, sumsq_out_stride};
+    g_gemv_hyper = {single, streams, count, mix, give, take};
+    const int status = gemv_checked(x, ldx, w, ldw, streams, n, m, n, k, kGemvHyper, nullptr, 0, nullptr, 0, nullptr, norm, stream);
+    g_gemv_hyper = {};
+    return status;
 }

@@ -213,9 +213,14 @@ class Model:
             if position + 1 < len(blocks) and not self.order[position + 1].before:
                 entry = getattr(blocks[position + 1], "entry_norm", None)
                 stream.upcoming = entry() if entry is not None else None
+            stream.reader = None
+            if position + 1 < len(blocks) and not self.order[position + 1].before:
+                reader = getattr(blocks[position + 1], "entry_reader", None)
+                stream.reader = reader(step) if reader is not None else None
             layer.block.run(stream, step)
         stream.after_layer = None
         stream.upcoming = None
+        stream.reader = None
         if n_logits == 0:
             stream.prepared = None
             return

@@ -106,6 +106,8 @@ _SIGNATURES = {
     "celeg_gemv_gate_constants": [c_float, c_float, c_float],
     "celeg_gemv_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                         c_void_p, c_longlong, c_void_p, c_void_p],
+    "celeg_gemv_hyper": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                         c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
     "celeg_gemv_prefetch_next": [c_void_p, c_longlong],
     "celeg_gemv_bf16_split_norm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                    c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_float, c_int,
@@ -696,6 +698,33 @@ def gemv_bf16(x, w: torch.Tensor, y: torch.Tensor, rows: int, mode: int = GEMV_S
         _ptr(next_weight) if prepare else None, _ptr(prepare.xw) if prepare else None,
         prepare.xw.stride(0) if prepare else 0, _ptr(prepare.sumsq) if prepare else None,
         prepare.sumsq.stride(0) if prepare else 0, _stream()))
+
+
+GEMV_MAX_STREAMS = 4
+
+
+def gemv_hyper(x, w: torch.Tensor, rows: int, streams: torch.Tensor, count: int, mix: torch.Tensor, give: torch.Tensor,
+               take: Optional[torch.Tensor], prepare: SplitNorm, next_weight: torch.Tensor, *,
+               single: Optional[torch.Tensor] = None, ahead: Optional[Tuple[int, int]] = None) -> None:
+    """y = x[:rows] @ w.T (at most 16 rows, w streamed once) mixed into ``count`` residual streams as :func:`hyper_connect`
+    does (x_t <- sum_s mix[s, t] x_s + give[t] y), and the norm of sum_t take[t] x_t with weight ``next_weight`` prepared in
+    ``prepare``. ``x`` may be a :class:`SplitNorm`."""
+    if ahead is not None and ahead[1] > 0:
+        if library().celeg_gemv_prefetch_next(ctypes.c_void_p(ahead[0]), ahead[1]) != 0:      # (no launch)
+            raise KernelLibraryError(library().celeg_last_error().decode("utf-8", "replace"))
+    n, k = w.shape
+    scaled = x if isinstance(x, SplitNorm) else None
+    operand = scaled.xw if scaled is not None else x
+    for tensor in (streams, mix, give, next_weight):
+        _need(tensor, torch.float32, "a tensor of gemv_hyper")
+    assert operand.shape[-1] == k and streams.numel() >= rows * count * n and mix.numel() == count * count
+    if prepare.partials != (n + 15) // 16 or prepare.sumsq.stride(0) < prepare.partials:
+        raise KernelLibraryError(f"a product of {n} columns writes {(n + 15) // 16} pieces of the sums, not {prepare.partials}")
+    _check(library().celeg_gemv_hyper(
+        _ptr(operand), operand.stride(0), _ptr(w), w.stride(0), rows, n, k, _ptr(single), _ptr(streams), count, _ptr(mix),
+        _ptr(give), _ptr(take), _ptr(scaled.sumsq) if scaled else None, scaled.partials if scaled else 0,
+        scaled.sumsq.stride(0) if scaled else 0, scaled.eps if scaled else 0.0, scaled.width if scaled else 0,
+        _ptr(next_weight), _ptr(prepare.xw), prepare.xw.stride(0), _ptr(prepare.sumsq), prepare.sumsq.stride(0), _stream()))
 
 
 TC_STORE, TC_STORE_F32, TC_SWIGLU = 0, 1, 2

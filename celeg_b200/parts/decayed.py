@@ -113,6 +113,9 @@ class Mamba2Mixer:
 
     ends_with_product = True      # forward() writes `out` last, with rt.linear
 
+    def takes_split_norm(self, step: StepContext) -> bool:
+        return self.rt.takes_split_norm(step.tokens, self.w_in)
+
     def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
         rt, t, b = self.rt, step.tokens, self.binding
         rt.linear(x, self.w_in, self.projected, t)
@@ -192,6 +195,9 @@ class GatedLinearAttentionMixer:
         self.binding = binding
 
     ends_with_product = True      # forward() writes `out` last, with rt.linear
+
+    def takes_split_norm(self, step: StepContext) -> bool:
+        return self.rt.takes_split_norm(step.tokens, self.w_in)
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> None:
         rt, t, b, qk, vw = self.rt, step.tokens, self.binding, self.qk_width, self.v_width

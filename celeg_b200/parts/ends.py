@@ -23,6 +23,7 @@ from typing import Mapping
 import torch
 
 from .. import kernels
+from .norms import RmsNorm
 from .registry import register_part
 from .runtime import Runtime, StepContext
 
@@ -76,6 +77,9 @@ class NormHeadOutput:
         self.multiplier = float(params.get("multiplier", 1.0))
         cap = params.get("softcap")
         self.softcap = float(cap) if cap else None        # logits <- cap * tanh(logits / cap)
+        if self.multiplier != 1.0 and isinstance(self.norm, RmsNorm):      # (the norm's weight is a scale: one for both)
+            self.norm.weight.mul_(self.multiplier)
+            self.multiplier = 1.0
         self.normed = rt.scratch("model.final_normed", int(self.head.shape[1]))
 
     def next_norm(self, step: StepContext, n_logits: int):

@@ -10,7 +10,9 @@
 
 All streams begin as the embedding row, which stays where the input part wrote it until the first sublayer's output is
 mixed in. What lies between two sublayers (mixing an output in, the next weighted sum, its norm) is one launch
-(csrc/hyper_connections.cu); the last norm's reader gets the norm of the streams' sum for the rows it wants.
+(csrc/hyper_connections.cu); the last norm's reader gets the norm of the streams' sum for the rows it wants. In steps of few
+rows on the bfloat16 path that launch falls away too where a sublayer ends in a product and the next one begins with one:
+the product mixes itself in and prepares the next norm (csrc/gemv_bf16.cu), as it does for one stream.
 """
 from __future__ import annotations
 
@@ -20,7 +22,7 @@ import torch
 
 from .. import kernels
 from .registry import register_part
-from .runtime import ResidualStream, Runtime, StepContext
+from .runtime import ResidualStream, Runtime, StepContext, _Sink
 
 
 class StreamCopies:
@@ -33,16 +35,52 @@ class StreamCopies:
         self.open = False
         self.single: Optional[torch.Tensor] = None       # the row that stands for every stream so far
         self.owed = None                                 # (connection, output, second output, both outputs' norms)
+        self.prepared = None                             # (connection or None, norm, SplitNorm) left by the last product
 
     def begin(self, stream: ResidualStream) -> None:
         """All streams become the stream's rows as they are."""
         if stream.pending is not None or stream.pending_b is not None or stream.prepared is not None:
             raise RuntimeError("the streams are opened from a stream that something is owed to")
-        self.open, self.single, self.owed = True, stream.residual, None
+        self.open, self.single, self.owed, self.prepared = True, stream.residual, None, None
 
     def read(self, connection: "HyperConnection", norm, out: torch.Tensor, rows: int) -> torch.Tensor:
-        """out = norm(sum_s take[s] x_s), what is owed mixed in for good."""
+        """out = norm(sum_s take[s] x_s), what is owed mixed in for good; or the split norm that the last product prepared
+        for exactly this reader."""
+        if self.prepared is not None:
+            return self._prepared_for(connection, norm)
         self._pass(out, rows, norm, connection.take, None)
+        return out
+
+    def _prepared_for(self, connection, norm):
+        prepared, self.prepared = self.prepared, None
+        if prepared[0] is not connection or prepared[1] is not norm:
+            raise RuntimeError("a norm was prepared for another reader than the one that asks")
+        return prepared[2]
+
+    def expect(self, stream: ResidualStream, buffer: torch.Tensor, connection: "HyperConnection", reader, rows: int) -> None:
+        """A sublayer with weights ``connection`` is about to write its output to ``buffer``; ``reader`` = (connection or
+        None, norm) of what reads the streams after it (None: it wants normalised rows)."""
+        rt = stream.rt
+        rt.sink = None
+        if reader is None or reader[1] is None or not rt.small_batch(rows) or self.count > kernels.GEMV_MAX_STREAMS:
+            return
+        halves = stream.split(reader[1], stream.pieces)
+        if halves is not None:
+            rt.sink = _Sink(buffer, reader[1], halves[0], halves[1], copies=self)
+            self.mixing, self.reader = connection, reader[0]
+
+    def take_product(self, x, weight: torch.Tensor, rows: int, sink: _Sink, ahead) -> None:
+        kernels.gemv_hyper(x, weight, rows, self.streams, self.count, self.mixing.mix, self.mixing.give,
+                           self.reader.take if self.reader is not None else None, sink.split, sink.weight, single=self.single,
+                           ahead=ahead)
+        self.single = None
+        self.prepared = (self.reader, sink.norm, sink.split)
+
+    def closing(self, norm, out: torch.Tensor, rows: int, gather: Optional[torch.Tensor] = None):
+        """norm(sum of the streams) of the rows (or the gathered ones) in ``out``, or as the last product prepared it."""
+        if self.prepared is not None and gather is None:
+            return self._prepared_for(None, norm)
+        self.total(out, rows, norm=norm, gather=gather)
         return out
 
     def owe(self, connection: "HyperConnection", y: torch.Tensor, second: Optional[torch.Tensor] = None, norms=None) -> None:
@@ -103,16 +141,33 @@ class HyperResidual:
         self.output = rt.scratch("block.output", hidden, torch.float32)
         self.delta = rt.scratch("block.delta_a", hidden)
 
-    def _sublayer(self, connection, norm, part, copies: StreamCopies, step: StepContext) -> None:
+    def _sublayer(self, connection, norm, part, reader, stream: ResidualStream, copies: StreamCopies,
+                  step: StepContext) -> None:
         x = copies.read(connection, norm, self.normed, step.tokens)
+        self.rt.sink = None
         pair = part.forward_normed_pair(x, step) if hasattr(part, "forward_normed_pair") else None
         if pair is not None:
             first, second, norms = pair
             copies.owe(connection, first, second, norms)
             return
-        output = self.output if getattr(part, "ends_with_product", False) else self.delta
-        part.forward(x, output, step)
-        copies.owe(connection, output)
+        if not getattr(part, "ends_with_product", False):
+            part.forward(x, self.delta, step)
+            copies.owe(connection, self.delta)
+            return
+        copies.expect(stream, self.output, connection, reader, step.tokens)
+        part.forward(x, self.output, step)
+        sink, self.rt.sink = self.rt.sink, None
+        if sink is None or not sink.used:
+            copies.owe(connection, self.output)
+
+    @staticmethod
+    def _takes_split(part, step: StepContext) -> bool:
+        takes = getattr(part, "takes_split_norm", None)
+        return takes is not None and takes(step)
+
+    def entry_reader(self, step: StepContext):
+        """(connection, norm) that the streams are read through first, if that reader takes a split norm."""
+        return (self.mixer_connection, self.mixer_norm) if self._takes_split(self.mixer, step) else None
 
     def run(self, stream: ResidualStream, step: StepContext) -> None:
         copies = stream.copies
@@ -122,6 +177,10 @@ class HyperResidual:
             copies.begin(stream)
         if copies.count != self.mixer_connection.streams:
             raise RuntimeError(f"a block of {self.mixer_connection.streams} streams among blocks of {copies.count}")
-        self._sublayer(self.mixer_connection, self.mixer_norm, self.mixer, copies, step)
-        if self.ffn is not None:
-            self._sublayer(self.ffn_connection, self.ffn_norm, self.ffn, copies, step)
+        after = stream.reader if stream.reader is not None else (None, stream.after_layer)
+        if self.ffn is None:
+            self._sublayer(self.mixer_connection, self.mixer_norm, self.mixer, after, stream, copies, step)
+            return
+        between = (self.ffn_connection, self.ffn_norm) if self._takes_split(self.ffn, step) else None
+        self._sublayer(self.mixer_connection, self.mixer_norm, self.mixer, between, stream, copies, step)
+        self._sublayer(self.ffn_connection, self.ffn_norm, self.ffn, after, stream, copies, step)

@@ -613,6 +613,9 @@ class PreparedAttentionMixer(PagedAttentionKernels):
             kernels.sigmoid_gate(self.attended, self.projected[:, at:at + self.gate_width], t, self.heads * self.value_dim,
                                  self.value_dim if self.gate_per_head else 1)
 
+    def takes_split_norm(self, step: StepContext) -> bool:
+        return self.rt.takes_split_norm(step.tokens, self.w_qkv)
+
     def forward_without_bias(self, x: torch.Tensor, out: torch.Tensor, step: StepContext) -> Optional[torch.Tensor]:
         """forward() into a float32 ``out`` without the output projection's bias, which is returned (or None) for a
         caller that adds it in a pass of its own."""
@@ -658,6 +661,9 @@ class SideBySideMixer:
         if "left_norm" in weights or "right_norm" in weights:
             self.norms = (rt.vector(weights["left_norm"]).mul_(self.left_scale),
                           rt.vector(weights["right_norm"]).mul_(self.right_scale), float(params["eps"]))
+
+    def takes_split_norm(self, step: StepContext) -> bool:
+        return all(hasattr(child, "takes_split_norm") and child.takes_split_norm(step) for child in (self.left, self.right))
 
     @staticmethod
     def _run(child, x, out, step):

@@ -15,11 +15,13 @@ LIBRARY_ROW_STEP = 64        # row counts of library products are rounded up to 
 
 
 class _Sink:
-    """Where a part is about to leave its output, and the norm that will read the stream next."""
-    __slots__ = ("buffer", "norm", "weight", "split", "used")
+    """Where a part is about to leave its output, and the norm that will read the stream next. ``copies``: the stream is
+    several streams (parts/hyper_connections.py), which take the product themselves."""
+    __slots__ = ("buffer", "norm", "weight", "split", "used", "copies")
 
-    def __init__(self, buffer, norm, weight, split):
+    def __init__(self, buffer, norm, weight, split, copies=None):
         self.buffer, self.norm, self.weight, self.split, self.used = buffer, norm, weight, split, False
+        self.copies = copies
 
 
 class ResidualStream:
@@ -44,6 +46,9 @@ class ResidualStream:
         # (norm, buffer) that the block after the one being run will ask for first, for every row of the step; a
         # stream part that runs after a block may write that norm's output itself and say so in ``ready``
         self.upcoming = None
+        # blocks over several streams: the connection and norm that the next block reads through first, if its mixer takes
+        # a split norm
+        self.reader = None
         self.ready = None
         # blocks whose sublayers read the stream itself: its rows in the activation type (on the float32 path the
         # stream's own), whether they are those of the stream as it is now, and whether the first block wants them
@@ -63,6 +68,7 @@ class ResidualStream:
         self.prepared = None
         self.after_layer = None
         self.upcoming = None
+        self.reader = None
         self.ready = None
         self.rows_current = False
         self.rt.sink = None
@@ -112,8 +118,7 @@ class ResidualStream:
         ``gather`` what was pending is added for good. Returns ``out``, or the split norm that the
         last product prepared for exactly this norm."""
         if self.copies is not None and self.copies.open:
-            self.copies.total(out, rows, norm=norm, gather=gather)
-            return out
+            return self.copies.closing(norm, out, rows, gather)
         if self.prepared is not None:
             prepared_norm, split = self.prepared
             self.prepared = None
@@ -317,6 +322,10 @@ class Runtime:
             kernels.gemm_f32(x, weight, out, rows)
         elif kernels.gemv_supported(rows, operand, weight):
             sink = self.sink
+            if sink is not None and sink.copies is not None and out is sink.buffer:
+                sink.copies.take_product(x, weight, rows, sink, self._ahead(weight))      # mixed into the streams here
+                sink.used = True
+                return
             if sink is not None and out is sink.buffer and weight.shape[0] == self.sink_residual.shape[1]:
                 # the product that ends a part: added to the stream here, and the next norm prepared
                 kernels.gemv_bf16(x, weight, self.sink_residual, rows, kernels.GEMV_ADD_RESIDUAL,
