@@ -230,7 +230,7 @@ def attention_case(heads, groups, dim, spans, last, seed, one_distance=None):
 KERNELS = ["generic", "prefill", "tcgen05", "decode"]
 
 
-def run_attention(kind, paged, queries, heads, groups, dim, scale, window, bias, sinks, dtype):
+def run_attention(kind, paged, queries, heads, groups, dim, scale, window, bias, sinks, dtype, softcap=None):
     k = kernels()
     positions, token_span, span_begin, table = paged.device()
     tokens = paged.tokens
@@ -241,15 +241,18 @@ def run_attention(kind, paged, queries, heads, groups, dim, scale, window, bias,
     spans = len(paged.spans)
     if kind == "generic":
         k.attention_generic(q, heads * dim, out, paged.k, paged.v, positions, token_span, table, tokens, heads, groups, dim,
-                            paged.page_tokens, window, scale, paged.flag, sinks=sinks_dev, distance_bias=bias_dev)
+                            paged.page_tokens, window, scale, paged.flag, sinks=sinks_dev, distance_bias=bias_dev,
+                            softcap=softcap)
     elif kind == "prefill":
         k.attention_prefill(q, heads * dim, out, paged.k, paged.v, positions, span_begin, table, tokens, spans, heads,
-                            groups, dim, paged.page_tokens, window, scale, paged.flag, sinks=sinks_dev, distance_bias=bias_dev)
+                            groups, dim, paged.page_tokens, window, scale, paged.flag, sinks=sinks_dev, distance_bias=bias_dev,
+                            softcap=softcap)
     elif kind == "tcgen05":
         tiles = sum(-(-new // 128) for _, new in paged.spans)
         k.attention_prefill_tcgen05(q, heads * dim, out, paged.k, paged.v, positions, span_begin, table, tokens, spans,
                                     tiles, heads, groups, dim, paged.page_tokens, window, scale, paged.flag,
-                                    sinks=sinks_dev, distance_bias=bias_dev)
+                                    sinks=sinks_dev, distance_bias=bias_dev,
+                            softcap=softcap)
     else:
         chunk, splits = 128, 8
         partial_o = torch.zeros(tokens * heads * splits * dim, dtype=torch.float32, device=DEVICE)
@@ -257,7 +260,8 @@ def run_attention(kind, paged, queries, heads, groups, dim, scale, window, bias,
         counters = torch.zeros(tokens * groups, dtype=torch.int32, device=DEVICE)
         k.attention_decode(q, heads * dim, out, paged.k, paged.v, positions, token_span, table, tokens, heads, groups, dim,
                            paged.page_tokens, window, scale, chunk, splits, partial_o, partial_ml, counters, paged.flag,
-                           sinks=sinks_dev, distance_bias=bias_dev)
+                           sinks=sinks_dev, distance_bias=bias_dev,
+                            softcap=softcap)
     torch.cuda.synchronize()
     assert int(paged.flag.item()) == 0
     return out.float().cpu().numpy().reshape(tokens, heads, dim).astype(np.float64)
