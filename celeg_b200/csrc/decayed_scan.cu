@@ -16,7 +16,8 @@
 // so all chunks are worked on side by side but for one element-wise walk over their states:
 //
 //   prepare   what the chunk's tokens do to one another, and the vectors q P(1..), k P(..n). Scalar: the running sums of
-//             the decays' logarithms; products of decays are exponentials of differences of those. Channel: the 64 tokens
+//             the decays' logarithms, each as two floats (a decay of almost nothing makes a sum large beside the differences
+//             that later tokens need); products of decays are exponentials of differences of those. Channel: the 64 tokens
 //             are eight blocks of eight, and within a block queries and keys are taken to its middle, q_i P(5..i) or
 //             q_i / P(i+1..4), k_j P(j+1..4) or k_j / P(5..j): at most four decays are divided by, and as a decay below
 //             1e-8 counts as 1e-8 (the old state's share is then below float32's rounding) that stays within range. The
@@ -54,11 +55,18 @@ __global__ void chunk_plan_kernel(const int* span_begin, int spans, int chunk, i
 }
 
 // ------------------------------------------------------------------------------------------------- prepare, scalar
-// cum[t, h]: the sum of the decays' logarithms from the chunk's first token through t; dt[t, h]. A block takes 8 heads of a
-// chunk: a warp a head, two neighbouring tokens a lane, the running sum by shuffles.
+__device__ __forceinline__ float2 two_floats(double x) {
+    const float high = (float)x;
+    return make_float2(high, (float)(x - (double)high));
+}
+
+// cum[t, h]: the sum of the decays' logarithms from the chunk's first token through t, a float and what it leaves of the double
+// that is summed in; dt[t, h]. A block takes 8 heads of a chunk: a warp a head, two neighbouring tokens a lane, the running
+// sum by shuffles.
 __global__ void __launch_bounds__(256) scalar_decay_kernel(const float* raw, int stride, const float* bias, const float* a_log,
-                                                           const int* chunk_begin, float* cum, float* dt, int heads) {
-    __shared__ float raw_s[kChunk][9], cum_s[kChunk][9], dt_s[kChunk][9];
+                                                           const int* chunk_begin, float2* cum, float* dt, int heads) {
+    __shared__ float raw_s[kChunk][9], dt_s[kChunk][9];
+    __shared__ float2 cum_s[kChunk][9];
     chain_release();
     chain_wait();
     const int h0 = blockIdx.x * 8;
@@ -73,17 +81,17 @@ __global__ void __launch_bounds__(256) scalar_decay_kernel(const float* raw, int
     if (h0 + warp < heads) {
         const float rate = expf(a_log[h0 + warp]), b = bias[h0 + warp];
         const float first = softplus_of(raw_s[2 * lane][warp] + b), second = softplus_of(raw_s[2 * lane + 1][warp] + b);
-        const float x = -rate * first, y = -rate * second;
-        float sum = x + y;
+        const double x = -rate * first, y = -rate * second;      // (products of floats)
+        double sum = x + y;
 #pragma unroll
         for (int offset = 1; offset < 32; offset <<= 1) {
-            const float below = __shfl_up_sync(0xffffffffu, sum, offset);
+            const double below = __shfl_up_sync(0xffffffffu, sum, offset);
             if (lane >= offset) sum += below;
         }
-        const float up = __shfl_up_sync(0xffffffffu, sum, 1);
-        const float before = lane > 0 ? up : 0.0f;
-        cum_s[2 * lane][warp] = before + x;
-        cum_s[2 * lane + 1][warp] = (before + x) + y;
+        const double up = __shfl_up_sync(0xffffffffu, sum, 1);
+        const double before = lane > 0 ? up : 0.0;
+        cum_s[2 * lane][warp] = two_floats(before + x);
+        cum_s[2 * lane + 1][warp] = two_floats(before + x + y);
         dt_s[2 * lane][warp] = first;
         dt_s[2 * lane + 1][warp] = second;
     }
@@ -94,6 +102,11 @@ __global__ void __launch_bounds__(256) scalar_decay_kernel(const float* raw, int
         cum[(size_t)(begin + t) * heads + h0 + h] = cum_s[t][h];
         dt[(size_t)(begin + t) * heads + h0 + h] = dt_s[t][h];
     }
+}
+
+// exp of the difference of two such sums
+__device__ __forceinline__ float decay_between(const float2& later, const float2& earlier) {
+    return expf((later.x - earlier.x) + (later.y - earlier.y));
 }
 
 // A tile of 64 x 64 floats into shared memory: rows r < rows of `src` (`stride` apart) times scale(r), columns c < columns;
@@ -313,7 +326,7 @@ static int launch_channel_prepare(const ChannelPrepareArgs& args, int chunks, cu
 struct ChunkArgs {
     const float* q; int q_stride; const float* k; int k_stride;        // channel: prepared; scalar: as projected, shared
     const float* v; int v_stride;
-    const float* cum; const float* dt;       // scalar: [tokens, heads]
+    const float2* cum; const float* dt;      // scalar: [tokens, heads]
     const float* total;                      // channel: [chunks, heads * dim]
     const float* products;                   // channel: per head; scalar: per group of heads
     const float* direct;                     // scalar: [heads], the values' share of the read-out, or null
@@ -340,7 +353,7 @@ __global__ void __launch_bounds__(256) chunk_states_kernel(const ChunkArgs p) {
     if (!CHANNEL) {
         if (threadIdx.x < count) {
             const size_t t = (size_t)(begin + threadIdx.x) * p.heads + head;
-            w_s[threadIdx.x] = p.dt[t] * expf(p.cum[(size_t)(begin + count - 1) * p.heads + head] - p.cum[t]);
+            w_s[threadIdx.x] = p.dt[t] * decay_between(p.cum[(size_t)(begin + count - 1) * p.heads + head], p.cum[t]);
         }
         __syncthreads();
     }
@@ -420,7 +433,7 @@ __global__ void __launch_bounds__(128) chunk_carry_kernel(const ChunkArgs p, flo
         if (!CHANNEL) {
 #pragma unroll
             for (int i = 0; i < kAhead; ++i)
-                if (c0 + i < last) keep[i] = p.cum[(size_t)ends[i] * p.heads + head];
+                if (c0 + i < last) keep[i] = p.cum[(size_t)ends[i] * p.heads + head].x;
         }
 #pragma unroll
         for (int i = 0; i < kAhead; ++i) {
@@ -465,7 +478,8 @@ template <bool CHANNEL>
 __global__ void __launch_bounds__(256, 4) chunk_outputs_kernel(const ChunkArgs p) {
     __shared__ __align__(16) float a_s[kChunk][kPitch];
     __shared__ __align__(16) float b_s[kChunk][kPitch];
-    __shared__ float cum_s[kChunk], dt_s[kChunk];
+    __shared__ float2 cum_s[kChunk];
+    __shared__ float dt_s[kChunk];
     chain_release();
     chain_wait();
     const int chunk = blockIdx.z, head = blockIdx.y, c0 = blockIdx.x * kChunk;
@@ -475,7 +489,7 @@ __global__ void __launch_bounds__(256, 4) chunk_outputs_kernel(const ChunkArgs p
     if (!CHANNEL) {
         if (threadIdx.x < kChunk) {
             const size_t t = (size_t)(begin + threadIdx.x) * p.heads + head;
-            cum_s[threadIdx.x] = threadIdx.x < count ? p.cum[t] : 0.0f;
+            cum_s[threadIdx.x] = threadIdx.x < count ? p.cum[t] : make_float2(0.0f, 0.0f);
             dt_s[threadIdx.x] = threadIdx.x < count ? p.dt[t] : 0.0f;
         }
         __syncthreads();
@@ -496,7 +510,7 @@ __global__ void __launch_bounds__(256, 4) chunk_outputs_kernel(const ChunkArgs p
             for (int i = 0; i < 4; ++i) {
                 const bool seen = c + i <= r && r < count;
                 if (CHANNEL) v[i] = seen ? v[i] : 0.0f;
-                else v[i] = seen ? v[i] * expf(cum_s[r] - cum_s[c + i]) * dt_s[c + i] : 0.0f;
+                else v[i] = seen ? v[i] * decay_between(cum_s[r], cum_s[c + i]) * dt_s[c + i] : 0.0f;
             }
             *reinterpret_cast<float4*>(&a_s[r][c]) = make_float4(v[0], v[1], v[2], v[3]);
         }
@@ -519,7 +533,7 @@ __global__ void __launch_bounds__(256, 4) chunk_outputs_kernel(const ChunkArgs p
         const float* q_src = p.q + (size_t)begin * p.q_stride + (size_t)group * p.dim + e0;
         if (CHANNEL) load_tile(a_s, q_src, p.q_stride, count, p.dim - e0, by_fours(p.q, p.q_stride, p.dim), NoScale());
         else load_tile(a_s, q_src, p.q_stride, count, p.dim - e0, by_fours(p.q, p.q_stride, p.dim),
-                       [&](int r) { return expf(cum_s[r]); });
+                       [&](int r) { return expf(cum_s[r].x); });
         load_tile(b_s, state + (size_t)e0 * p.vdim + c0, p.vdim, p.dim - e0, p.vdim - c0, by_fours(p.states, p.vdim, p.dim * p.vdim),
                   NoScale());
         __syncthreads();
@@ -746,10 +760,10 @@ CELEG_API int celeg_channel_decay_scan(const float* q, int q_stride, const float
 }
 
 // The scalar form: q and k have `groups` heads of dim that heads / groups heads of v share; raw: the steps before bias and
-// softplus, head h in column h. Scratch: cum, dt [tokens, heads], products [chunks, groups, 64, 64], states as above.
+// softplus, head h in column h. Scratch: cum (two floats each), dt [tokens, heads], products [chunks, groups, 64, 64], states as above.
 CELEG_API int celeg_scalar_decay_scan(const float* q, int q_stride, const float* k, int k_stride, const float* v, int v_stride,
                                       const float* raw, int raw_stride, const float* dt_bias, const float* a_log,
-                                      const float* direct, float* cum, float* dt, float* products, float* states, float* out,
+                                      const float* direct, float2* cum, float* dt, float* products, float* states, float* out,
                                       float* state, long long slot_stride, const int* span_slot, const int* plan,
                                       int max_chunks, int spans, int chunks, int heads, int groups, int dim, int vdim,
                                       cudaStream_t stream) {

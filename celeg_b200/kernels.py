@@ -1386,7 +1386,9 @@ def scalar_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: to
                       span_slot: torch.Tensor, plan: torch.Tensor, max_chunks: int, spans: int, chunks: int, heads: int,
                       groups: int, dim: int, vdim: int) -> None:
     """S <- exp(-exp(a_log) dt) S + dt k v^T, o = S^T q + direct v with dt = softplus(raw + dt_bias) along the step's spans;
-    heads / groups heads share queries and keys (csrc/decayed_scan.cu)."""
+    heads / groups heads share queries and keys (csrc/decayed_scan.cu). Scratch: ``cum`` [tokens, 2 heads], ``dt`` [tokens,
+    heads]."""
+    assert cum.is_contiguous() and cum.shape[1] == 2 * heads and dt.is_contiguous() and dt.shape[1] == heads
     for tensor in (q, k, v, raw, dt_bias, a_log, cum, dt, products, states, out, state):
         assert tensor.dtype == torch.float32 and tensor.stride(-1) == 1
     assert out.is_contiguous() and out.shape[1] == heads * vdim and states.numel() >= chunks * heads * dim * vdim

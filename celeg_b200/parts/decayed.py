@@ -97,7 +97,7 @@ class Mamba2Mixer:
         chunks = self.spans.max_chunks
         self.projected = rt.scratch("recurrent.proj", int(self.w_in.shape[0]), torch.float32)
         self.convolved = rt.scratch("recurrent.conv", self.channels, torch.float32)
-        self.cum = rt.scratch("decay.cum", self.heads, torch.float32)
+        self.cum = rt.scratch("decay.cum", 2 * self.heads, torch.float32)
         self.dt = rt.scratch("decay.dt", self.heads, torch.float32)
         self.products = rt.flat_scratch("decay.products", chunks * self.groups * self.spans.tokens ** 2, torch.float32)
         self.states = rt.flat_scratch("decay.states", chunks * self.state_elements, torch.float32)

@@ -235,7 +235,8 @@ def test_the_scan_and_the_decoding_step_with_a_decay_a_channel(heads, dim, vdim,
 
 @pytest.mark.parametrize("lengths", LENGTHS)
 @pytest.mark.parametrize("heads,groups,dim,vdim", [(4, 2, 8, 4), (3, 1, 5, 7), (4, 4, 64, 64), (6, 2, 130, 72), (8, 1, 16, 33)])
-def test_the_scan_and_the_decoding_step_with_a_decay_a_token(heads, groups, dim, vdim, lengths):
+@pytest.mark.parametrize("forgets", [False, True])
+def test_the_scan_and_the_decoding_step_with_a_decay_a_token(heads, groups, dim, vdim, lengths, forgets):
     k = kernels()
     rng = np.random.default_rng(dim + 7 * len(lengths))
     elements = heads * dim * vdim
@@ -244,6 +245,14 @@ def test_the_scan_and_the_decoding_step_with_a_decay_a_token(heads, groups, dim,
     rows = rng.normal(size=(t, 2 * qk + vw + heads + 3)).astype(np.float32)
     dt_bias, a_log = rng.uniform(-4.0, 2.0, size=heads).astype(np.float32), rng.uniform(-3.0, 2.5, size=heads).astype(np.float32)
     direct = rng.normal(size=heads).astype(np.float32)
+    if forgets:
+        # tokens whose step is so long that nothing before them is left, among tokens that keep almost everything: the
+        # running sums are large beside the differences that the later tokens need
+        a_log[:] = rng.uniform(-1.0, 2.0, size=heads)
+        dt_bias[:] = -6.0
+        rows[1::29, 2 * qk + vw:2 * qk + vw + heads] = 3000.0
+        rows[1::29, vw:vw + qk] = 0.0                        # (and they write nothing)
+        direct[:] = 0.0
     v, key, q, raw = (f32(rows[:, a:b]) for a, b in ((0, vw), (vw, vw + qk), (vw + qk, vw + 2 * qk), (vw + 2 * qk, vw + 2 * qk + heads)))
     step = plain.softplus(raw + f32(dt_bias))
     decays = np.exp(-np.exp(f32(a_log)) * step)
@@ -262,12 +271,15 @@ def test_the_scan_and_the_decoding_step_with_a_decay_a_token(heads, groups, dim,
     chunks = t // k.chunk_tokens() + spans.spans + 1
     plan = torch.zeros(chunks + spans.spans + 2, dtype=torch.int32, device=DEVICE)
     buffers = [torch.zeros(size, dtype=torch.float32, device=DEVICE) for size in
-               ((t, heads), (t, heads), chunks * groups * 4096, chunks * elements, (t, vw))]
+               ((t, 2 * heads), (t, heads), chunks * groups * 4096, chunks * elements, (t, vw))]
     state = gpu(spans.state)
     k.chunk_plan(spans.dev["span_begin"], spans.spans, chunks, plan)
     k.scalar_decay_scan(*views, gpu(dt_bias), gpu(a_log), gpu(direct), *buffers, state, spans.state.shape[1], spans.dev["span_slot"],
                         plan, chunks, spans.spans, chunks - 1, heads, groups, dim, vdim)
     close(buffers[-1], want, 1e-5, "read-outs of the scan")
+    if forgets:                                              # every token by its own measure
+        size = np.abs(want).max(1, keepdims=True) + 1e-4
+        close(buffers[-1] / gpu(size), want / size, 3e-5, "read-outs of the scan, token by token")
     close(state, want_state, 4e-6, "states after the scan")
     if max(lengths) == 1:
         state, out = gpu(spans.state), torch.zeros((t, vw), dtype=torch.float32, device=DEVICE)
